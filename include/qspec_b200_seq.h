@@ -174,6 +174,11 @@ typedef struct qspec_window_attn_args {
   const float* sink; const void* gate; int gate_ld;
   void* out; const int* meta; int ntok, H, G, window, cap; float scale;
   int gate_per_head;   /* 0: gate[t, h * DV + d] as above; 1: one gate per head, gate[t, h] (gate_ld >= H) */
+  int keep_first;      /* > 0: the first keep_first positions stay visible to every later token (a token sees j when i - j < window or
+                          j < keep_first) and their ring rows are never reused: row = j for j < cap, otherwise keep_first +
+                          (j - keep_first) % (cap - keep_first). cap >= keep_first + window - 1 + (tokens of one sequence in a step). */
+  long long out_tok_stride;   /* elements from one token's output row to the next; 0: H * DV */
+  float out_scale;     /* factor on the output; 0: one */
 } qspec_window_attn_args;
 int qspec_seq_window_attention(const qspec_window_attn_args* args, int dtype, void* stream);
 
@@ -246,11 +251,11 @@ int qspec_seq_lightning(const void* p, int ld, const float* decay, const float* 
  * Scores s = softmax(z[0:R]) (score_fn 0) or sigmoid(z[0:R]) (score_fn 1); choice = s + correction (NULL: zeros). The R
  * experts form n_groups equal groups of neighbours; a group's score is the sum of its group_top largest choice scores; only
  * experts of the keep_groups best groups can be chosen (n_groups <= 1: no limit). The `top` largest remaining choices (lowest
- * index among equals) -> idx, weight = scale * s of the chosen. extra[t, x] = sigmoid(z[R + x]) for the n_extra gate rows
+ * index among equals) -> idx, weight = scale * s of the chosen, divided by (sum of the chosen s) + 1e-20 if normalize. extra[t, x] = sigmoid(z[R + x]) for the n_extra gate rows
  * (extra float32 [ntok, extra_ld]). R + n_extra <= 1024, top <= 32. */
 int qspec_moe_route_grouped(const void* h, const float* router_w, const float* correction, int* idx, float* weight, float* extra,
                             int extra_ld, int ntok, int W, int R, int top, int score_fn, int n_groups, int keep_groups,
-                            int group_top, float scale, int n_extra, int dtype, void* stream);
+                            int group_top, float scale, int normalize, int n_extra, int dtype, void* stream);
 
 /* Softmax attention of ONE prompt portion on the tensor cores, tile form (bfloat16): the ntok tokens are consecutive positions
  * pos0 .. pos0 + ntok - 1 of the sequence in slot `slot` (args->meta is not read). A CTA takes 64 tokens and one head and reads
@@ -332,6 +337,69 @@ int qspec_seq_glu_clamp(const void* gu, int ld, void* out, int ntok, int F, floa
 
 /* a <- s * a, n float32 values. */
 int qspec_seq_scale_f32(float* a, long long n, float s, void* stream);
+
+/* ---- norm without statistics, heads prepared from the projection, delta rule with channel decays, logit soft cap ---- */
+
+/* Residual sum and a tanh norm of the result in one launch:
+ *   r = x_in + mult * (sum_p y_w[t, p] * y[t, p, :] + y_bias)     (y NULL: r = x_in; y_w NULL: ones; y_bias float32 [W] or NULL)
+ *   out = tanh(alpha * r) * w + b
+ * r goes to x_out (float32, may alias x_in, may be NULL), the norm to out (activation type, may be NULL). y has element type
+ * y_dtype: the activation type or float32. */
+int qspec_seq_residual_tanh(const float* x_in, float* x_out, const void* y, int y_parts, long long y_part_stride,
+                            long long y_tok_stride, const float* y_w, const float* y_bias, float mult, float alpha, const float* w,
+                            const float* b, void* out, int ntok, int W, int y_dtype, int dtype, void* stream);
+
+/* a <- cap * tanh(a / cap), n float32 values. */
+int qspec_seq_softcap_f32(float* a, long long n, float cap, void* stream);
+
+/* Attention heads from the projection. Row t of p (leading dimension ld) holds q (H x D) at column q_off, k (G x D) at k_off and v
+ * (G x DV) at v_off; v_off < 0: the values are the keys as projected (DV = D, no convolution). In this order:
+ *   conv_w (float32 [taps][C], C = H D + G D + G DV channels in the order q, k, v; NULL: none): x_t <- sum_j conv_w[j] x_(t-taps+1+j),
+ *     the rows before the step from tail (float32 [2][slots][taps - 1][C], read at `phase`, written at 1 - `phase`), zeros before
+ *     position 0; values go to the cache as they are now
+ *   norm_last 0: q, k <- x / sqrt(mean over D of x^2 + eps) * qn_w / kn_w (float32 [D], NULL: ones)
+ *   rotation of the first rot_dims entries, entry i with entry i + rot_dims / 2 by the angle pos * inv_freq[i], cosine and sine
+ *     times rot_amp
+ *   norm_last 1: the norm comes here instead
+ *   temp_every > 0: q <- q * (1 + temp_coef * ln(floor((pos + 1) / temp_every) + 1))
+ * qout float32 [ntok, H, D]; cache_k [slots, cap, G, D] and cache_v [slots, cap, G, DV] take ring row pos (keep_first as in
+ * qspec_window_attn_args). D, DV <= 1024. */
+typedef struct qspec_head_prep_args {
+  const void* p; int ld, q_off, k_off, v_off;
+  const float* conv_w; int taps; float* tail; int slots;
+  const float* qn_w; const float* kn_w; int norm_last;
+  const float* inv_freq; int rot_dims; float rot_amp;
+  float temp_coef; int temp_every;
+  float* qout; void* cache_k; void* cache_v; int cap, keep_first;
+  const int* meta; int ntok, H, G, D, DV; float eps;
+} qspec_head_prep_args;
+int qspec_seq_head_prep(const qspec_head_prep_args* args, int dtype, void* stream);
+
+/* Gated delta rule with one decay per head and key channel, from the projection to the gated output. Row t of p (leading dimension
+ * ld, activation type): [q (G x D) | k (G x D) | v (H x DV)], and the H step-size logits at column beta_off (counted from p).
+ *   q, k, v <- silu(short causal convolution) (conv_w float32 [taps][C], C = 2 G D + H DV; tail as in qspec_head_prep_args)
+ *   q <- q / sqrt(sum q^2 + unit_eps) * q_mult, k likewise without q_mult
+ *   g = exp(-exp(A_log[h]) * softplus(decay[t, h D + d] + dt_bias[h D + d])), decay float32 with leading dimension decay_ld
+ *   S <- diag(g) S;  u = sigmoid(beta) (v - S^T k);  S <- S + k u^T;  o = S^T q     (head h uses query / key head h / (H / G))
+ *   out[t, h] = out_scale * o / sqrt(mean(o^2) + eps) * norm_w * sigmoid(gate[t, h DV + c])     (gate NULL: none)
+ * state: float32 [slots, H, D, DV], read at a segment's start (zero at position 0), written at its end. D <= 256.
+ * Segments of at most max_len tokens take a one-launch token form; the nlong longer ones a block form: block_rows int32 [nblocks]
+ * holds the batch row of the first token of every block of 16 tokens of those segments, in order, long_starts int32 [nlong] their
+ * first rows, long_block0 int32 [nlong] the index in block_rows of their first block. scratch (bytes from the query, 16-byte
+ * aligned) is needed for the block form only. seg_starts int32 [nseg]: the first rows of all segments. */
+typedef struct qspec_delta_channel_args {
+  const void* p; int ld, beta_off;
+  const float* conv_w; int taps; float* tail; int slots;
+  const float* decay; int decay_ld;
+  const float* A_log; const float* dt_bias; const float* norm_w;
+  const void* gate; int gate_ld;
+  float* state; void* out; int out_ld;
+  const int* meta; const int* seg_starts; int nseg, ntok, H, G, D, DV;
+  float unit_eps, q_mult, eps, out_scale;
+} qspec_delta_channel_args;
+size_t qspec_seq_delta_channel_scratch_bytes(int nblocks, int ntok, int H, int D, int DV);
+int qspec_seq_delta_channel(const qspec_delta_channel_args* args, const int* block_rows, int nblocks, const int* long_starts,
+                            const int* long_block0, int nlong, int max_len, void* scratch, size_t scratch_bytes, int dtype, void* stream);
 
 /* Arg max per row of float32 / bfloat16 logits [rows, V] (lowest index among equal maxima): int64 out. */
 int qspec_seq_argmax_rows(const void* logits, int rows, int V, long long row_stride, long long* out_idx, int dtype,

@@ -162,7 +162,7 @@ SEQ_SIGNATURES = {
     "qspec_seq_prompt_attention_mma": (c_int, [c_void_p, c_void_p, c_ll, c_int, c_int, c_int, c_int, c_void_p]),
     "qspec_seq_prompt_attention_mma_supported": (c_int, [c_int, c_int, c_int]),
     "qspec_moe_route_grouped": (c_int, [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
-                                        c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p]),
+                                        c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_void_p]),
     "qspec_seq_residual_norm_scaled": (c_int, [c_void_p, c_void_p, c_void_p, c_int, c_ll, c_ll, c_void_p, c_void_p, c_void_p, c_int,
                                                c_float, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_float, c_int, c_int,
                                                c_void_p]),
@@ -180,6 +180,12 @@ SEQ_SIGNATURES = {
     "qspec_seq_talking_attention": (c_int, [c_void_p, c_int, c_int, c_void_p]),
     "qspec_seq_glu_clamp": (c_int, [c_void_p, c_int, c_void_p, c_int, c_int, c_float, c_float, c_int, c_void_p]),
     "qspec_seq_scale_f32": (c_int, [c_void_p, c_ll, c_float, c_void_p]),
+    "qspec_seq_residual_tanh": (c_int, [c_void_p, c_void_p, c_void_p, c_int, c_ll, c_ll, c_void_p, c_void_p, c_float, c_float, c_void_p,
+                                        c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p]),
+    "qspec_seq_softcap_f32": (c_int, [c_void_p, c_ll, c_float, c_void_p]),
+    "qspec_seq_head_prep": (c_int, [c_void_p, c_int, c_void_p]),
+    "qspec_seq_delta_channel_scratch_bytes": (c_size_t, [c_int, c_int, c_int, c_int, c_int]),
+    "qspec_seq_delta_channel": (c_int, [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_size_t, c_int, c_void_p]),
 }
 
 
@@ -191,8 +197,31 @@ class WindowAttnArgs(ctypes.Structure):
                 ("v", c_void_p), ("v_slot_stride", c_ll), ("v_row_stride", c_int), ("v_head_stride", c_int), ("DV", c_int),
                 ("sink", c_void_p), ("gate", c_void_p), ("gate_ld", c_int),
                 ("out", c_void_p), ("meta", c_void_p), ("ntok", c_int), ("H", c_int), ("G", c_int), ("window", c_int),
-                ("cap", c_int), ("scale", c_float), ("gate_per_head", c_int)]
+                ("cap", c_int), ("scale", c_float), ("gate_per_head", c_int), ("keep_first", c_int), ("out_tok_stride", c_ll),
+                ("out_scale", c_float)]
 
+
+class HeadPrepArgs(ctypes.Structure):
+    """qspec_head_prep_args of include/qspec_b200_seq.h."""
+    _fields_ = [("p", c_void_p), ("ld", c_int), ("q_off", c_int), ("k_off", c_int), ("v_off", c_int),
+                ("conv_w", c_void_p), ("taps", c_int), ("tail", c_void_p), ("slots", c_int),
+                ("qn_w", c_void_p), ("kn_w", c_void_p), ("norm_last", c_int),
+                ("inv_freq", c_void_p), ("rot_dims", c_int), ("rot_amp", c_float),
+                ("temp_coef", c_float), ("temp_every", c_int),
+                ("qout", c_void_p), ("cache_k", c_void_p), ("cache_v", c_void_p), ("cap", c_int), ("keep_first", c_int),
+                ("meta", c_void_p), ("ntok", c_int), ("H", c_int), ("G", c_int), ("D", c_int), ("DV", c_int), ("eps", c_float)]
+
+
+class DeltaChannelArgs(ctypes.Structure):
+    """qspec_delta_channel_args of include/qspec_b200_seq.h."""
+    _fields_ = [("p", c_void_p), ("ld", c_int), ("beta_off", c_int),
+                ("conv_w", c_void_p), ("taps", c_int), ("tail", c_void_p), ("slots", c_int),
+                ("decay", c_void_p), ("decay_ld", c_int),
+                ("A_log", c_void_p), ("dt_bias", c_void_p), ("norm_w", c_void_p),
+                ("gate", c_void_p), ("gate_ld", c_int),
+                ("state", c_void_p), ("out", c_void_p), ("out_ld", c_int),
+                ("meta", c_void_p), ("seg_starts", c_void_p), ("nseg", c_int), ("ntok", c_int), ("H", c_int), ("G", c_int), ("D", c_int),
+                ("DV", c_int), ("unit_eps", c_float), ("q_mult", c_float), ("eps", c_float), ("out_scale", c_float)]
 
 
 class TalkingAttnArgs(ctypes.Structure):

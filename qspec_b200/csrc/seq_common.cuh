@@ -1,5 +1,5 @@
 // Helpers shared by the sequence-mixer kernel files: element conversion, the per-token row of the step table,
-// and 1- or 4-element vector loads / stores of float32 and bfloat16 rows.
+// 1- or 4-element vector loads / stores of float32 and bfloat16 rows, asynchronous copies, ring rows and activations.
 #pragma once
 #include "common.cuh"
 
@@ -53,5 +53,25 @@ template <int VEC> __device__ __forceinline__ void stv(__nv_bfloat16* p, const V
     *reinterpret_cast<uint2*>(p) = t;
   } else *p = __float2bfloat16_rn(r.v[0]);
 }
+
+
+// Row of a position in a per-slot ring of `cap` rows whose first `keep` rows are never reused: positions below `keep` stay where
+// they are, the others go round the remaining rows. keep = 0: position % cap.
+__device__ __forceinline__ int ring_row(int pos, int keep, int cap) { return pos < cap ? pos : keep + (pos - keep) % (cap - keep); }
+
+// 4-byte asynchronous copies into shared memory (both addresses on 4-byte boundaries)
+__device__ __forceinline__ void cp_async_4(float* smem_dst, const float* src) {
+  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;\n" ::"r"((uint32_t)__cvta_generic_to_shared(smem_dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;\n" ::: "memory"); }
+template <int N> __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;\n" ::"n"(N) : "memory"); }
+
+// 16-byte asynchronous copy into shared memory; `valid` false writes zeros and reads nothing
+__device__ __forceinline__ void cp_async_16z(void* smem_dst, const void* src, bool valid) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"((uint32_t)__cvta_generic_to_shared(smem_dst)), "l"(src),
+               "r"(valid ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ float silu_f(float z) { return z / (1.0f + expf(-z)); }
+__device__ __forceinline__ float softplus_f(float z) { return z > 20.f ? z : log1pf(expf(z)); }
 
 }  // namespace qspec

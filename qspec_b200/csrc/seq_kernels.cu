@@ -539,7 +539,7 @@ __global__ void __launch_bounds__(256) relu2_kernel(T* __restrict__ a, long long
 // Router: one CTA of 128 threads per token. Dot products by warp, then scores (softmax or sigmoid), group limits and top-k
 // by one warp. The last n_extra rows of the router matrix are gate rows: their sigmoid goes to `extra`.
 struct RouteOpts {
-  int score_fn, n_groups, keep_groups, group_top, n_extra, extra_ld;
+  int score_fn, n_groups, keep_groups, group_top, n_extra, extra_ld, normalize;
   float scale;
   float* extra;
 };
@@ -681,6 +681,7 @@ route_kernel(const T* __restrict__ h, const float* __restrict__ rw, const float*
     }
     __syncwarp();
   }
+  float chosen_sum = 0.f;
   for (int k = 0; k < top; ++k) {
     float bv = -INFINITY;
     int bi = 0x7fffffff;
@@ -696,9 +697,14 @@ route_kernel(const T* __restrict__ h, const float* __restrict__ rw, const float*
     if (lane == 0) {
       idx[(size_t)i * top + k] = bi;
       weight[(size_t)i * top + k] = z[bi] * ro.scale;
+      chosen_sum += z[bi];
       ch[bi] = -INFINITY;
     }
     __syncwarp();
+  }
+  if (ro.normalize && lane == 0) {                            // the chosen scores divided by their sum
+    const float d = chosen_sum + 1e-20f;
+    for (int k = 0; k < top; ++k) weight[(size_t)i * top + k] /= d;
   }
 }
 
@@ -1045,7 +1051,7 @@ extern "C" int qspec_seq_relu2(void* a, long long n, int dtype, void* stream) {
 
 static int route_any(const void* h, const float* router_w, const float* correction, int* idx, float* weight, int ntok, int W, int R, int top,
                      int chosen_only, int dtype, void* stream, const RouteOpts* opts = nullptr) {
-  RouteOpts ro = {0, 1, 1, 1, 0, 0, 1.0f, nullptr};
+  RouteOpts ro = {0, 1, 1, 1, 0, 0, 0, 1.0f, nullptr};
   if (opts) ro = *opts;
   QSPEC_REQUIRE(h && router_w && (correction || chosen_only || opts) && idx && weight, QSPEC_ERR_INVALID_ARG, "moe_route: null pointer");
   QSPEC_REQUIRE(ntok >= 0 && W > 0 && R > 0 && R + ro.n_extra <= 1024 && top >= 1 && top <= 32 && top <= R, QSPEC_ERR_UNSUPPORTED,
@@ -1070,9 +1076,9 @@ static int route_any(const void* h, const float* router_w, const float* correcti
 
 extern "C" int qspec_moe_route_grouped(const void* h, const float* router_w, const float* correction, int* idx, float* weight, float* extra,
                                        int extra_ld, int ntok, int W, int R, int top, int score_fn, int n_groups, int keep_groups,
-                                       int group_top, float scale, int n_extra, int dtype, void* stream) {
+                                       int group_top, float scale, int normalize, int n_extra, int dtype, void* stream) {
   QSPEC_REQUIRE(score_fn == 0 || score_fn == 1, QSPEC_ERR_INVALID_ARG, "moe_route_grouped: score function %d", score_fn);
-  RouteOpts ro = {score_fn, n_groups < 1 ? 1 : n_groups, n_groups < 1 ? 1 : keep_groups, group_top, n_extra, extra_ld, scale, extra};
+  RouteOpts ro = {score_fn, n_groups < 1 ? 1 : n_groups, n_groups < 1 ? 1 : keep_groups, group_top, n_extra, extra_ld, normalize ? 1 : 0, scale, extra};
   return route_any(h, router_w, correction, idx, weight, ntok, W, R, top, 0, dtype, stream, &ro);
 }
 

@@ -196,7 +196,7 @@ window_attn_kernel(const float* __restrict__ qa, long long qa_ts, long long qa_h
                    long long qb_ts, long long qb_hs, int DB, const T* __restrict__ kc, long long k_ss, int k_rs, int k_hs,
                    const T* __restrict__ vc, long long v_ss, int v_rs, int v_hs, int DV, const float* __restrict__ sink,
                    const T* __restrict__ gate, int gate_ld, int gate_per_head, T* __restrict__ out, const int* __restrict__ meta,
-                   int ntok, int H, int G, int window, int cap, float scale) {
+                   int ntok, int H, int G, int window, int cap, float scale, int keep, long long out_ts, float out_scale) {
   pdl_enter();
   extern __shared__ float sm_wa[];            // q [DK] | acc [4][DV]
   __shared__ float s_m[4], s_l[4];
@@ -211,20 +211,21 @@ window_attn_kernel(const float* __restrict__ qa, long long qa_ts, long long qa_h
   __syncthreads();
   const T* kbase = kc + (size_t)slot * k_ss + (size_t)g * k_hs;
   const T* vbase = vc + (size_t)slot * v_ss + (size_t)g * v_hs;
-  const int j0 = max(0, pos - window + 1);
+  // visible keys in order: the first nk positions (kept ones that the window has left behind), then the window from j0 on
+  const int j0 = max(0, pos - window + 1), nk = min(keep, j0), nkeys = nk + pos - j0 + 1;
   float m = -INFINITY, l = 0.f;
   float acc[NACC];
 #pragma unroll
   for (int a = 0; a < NACC; ++a) acc[a] = 0.f;
   // a warp takes runs of KU consecutive keys (every fourth run): KU independent rows in flight per iteration
   constexpr int KU = 4;
-  for (int j = j0 + warp * KU; j <= pos; j += 4 * KU) {
-    const int n = min(KU, pos - j + 1);
+  for (int j = warp * KU; j < nkeys; j += 4 * KU) {
+    const int n = min(KU, nkeys - j);
     const T* kr[KU];
     const T* vr[KU];
 #pragma unroll
     for (int u = 0; u < KU; ++u) {
-      const int r = (j + (u < n ? u : 0)) % cap;
+      const int ju = j + (u < n ? u : 0), r = ring_row(ju < nk ? ju : j0 + ju - nk, keep, cap);
       kr[u] = kbase + (size_t)r * k_rs;
       vr[u] = vbase + (size_t)r * v_rs;
     }
@@ -294,9 +295,9 @@ window_attn_kernel(const float* __restrict__ qa, long long qa_ts, long long qa_h
     float o = 0.f;
 #pragma unroll
     for (int w = 0; w < 4; ++w) o += sacc[w * DV + c] * f[w];
-    o *= inv;
+    o *= inv * out_scale;
     if (gate) o *= 1.0f / (1.0f + expf(-to_f(gate[(size_t)i * gate_ld + (gate_per_head ? (size_t)h : (size_t)h * DV + c)])));
-    out[((size_t)i * H + h) * DV + c] = from_f<T>(o);
+    out[(size_t)i * out_ts + (size_t)h * DV + c] = from_f<T>(o);
   }
 }
 
@@ -721,7 +722,8 @@ static int launch_window_attn(const qspec_window_attn_args* a, cudaStream_t st) 
   launch_pdl(window_attn_kernel<T, NACC, VEC>, dim3(a->ntok, a->H), dim3(128), smem, st, a->qa, a->qa_tok_stride, a->qa_head_stride, a->DA,
              a->qb, a->qb_tok_stride, a->qb_head_stride, a->DB, (const T*)a->k, a->k_slot_stride, a->k_row_stride, a->k_head_stride,
              (const T*)a->v, a->v_slot_stride, a->v_row_stride, a->v_head_stride, a->DV, a->sink, (const T*)a->gate, a->gate_ld, a->gate_per_head, (T*)a->out,
-             a->meta, a->ntok, a->H, a->G, a->window, a->cap, a->scale);
+             a->meta, a->ntok, a->H, a->G, a->window, a->cap, a->scale, a->keep_first,
+             a->out_tok_stride ? a->out_tok_stride : (long long)a->H * a->DV, a->out_scale != 0.f ? a->out_scale : 1.0f);
   QSPEC_CHECK_LAUNCH(1);
   return QSPEC_OK;
 }
@@ -740,7 +742,7 @@ extern "C" int qspec_seq_window_attention(const qspec_window_attn_args* a, int d
   QSPEC_REQUIRE(a && a->qa && a->k && a->v && a->out && a->meta && (a->DB == 0 || a->qb), QSPEC_ERR_INVALID_ARG,
                 "seq_window_attention: null pointer");
   QSPEC_REQUIRE(a->ntok >= 0 && a->H > 0 && a->G > 0 && a->H % a->G == 0 && a->DA > 0 && a->DB >= 0 && a->DV > 0 && a->DV <= 1024 &&
-                    a->DA + a->DB <= 8192 && a->window >= 1 && a->cap >= 1 && a->H <= 65535,
+                    a->DA + a->DB <= 8192 && a->window >= 1 && a->cap >= 1 && a->H <= 65535 && a->keep_first >= 0 && a->keep_first < a->cap,
                 QSPEC_ERR_UNSUPPORTED, "seq_window_attention: heads %d / %d, key size %d + %d (<= 8192), value size %d (<= 1024)", a->H,
                 a->G, a->DA, a->DB, a->DV);
   MIX_DTYPE_OK(dtype);

@@ -7,7 +7,7 @@
 //    which is what rules out a plain TMA tile). The warp-level form of the same product is kept for comparison.
 #include <cstdlib>
 #include <cstring>
-#include "common.cuh"
+#include "seq_common.cuh"
 #include "../../include/qspec_b200_seq.h"
 
 namespace qspec {
@@ -980,6 +980,7 @@ struct WinMma {
   const bf16* v; long long v_ss; int v_rs, v_hs;
   const float* sink; const bf16* gate; int gate_ld, gate_per_head;
   bf16* out; int out_hs; const int* meta; int ntok, H, G, window, cap; float scale; int token_rows;
+  int keep; long long out_ts; float out_scale;
 };
 
 // STREAM: key rows are loaded inside the product loop instead of a whole step ahead (long keys: the fragments of a step
@@ -1032,8 +1033,10 @@ __global__ void __launch_bounds__(128, 2) window_attn_mma_kernel(const WinMma a)
     while (r1 < 16 && s_tok[r1] >= 0 && s_seg[r1] == s_seg[r0]) ++r1;
     const int seg = s_seg[r0], slot = s_slot[r0];
     const int pmax = a.token_rows ? s_pos[r1 - 1] : s_pos[r0];
-    const int jlo = max(0, s_pos[r0] - a.window + 1);
-    const int nkeys = pmax - jlo + 1;
+    // keys in order: nk kept positions that the first row's window has left behind, then positions from jlo on
+    const int jlo = max(0, s_pos[r0] - a.window + 1), nk = min(a.keep, jlo);
+    const int nkeys = nk + pmax - jlo + 1;
+    auto key_row = [&](int jj) { return ring_row(jj < nk ? jj : jlo + jj - nk, a.keep, a.cap); };
     const bf16* kA = a.kA + (size_t)slot * a.kA_ss + (size_t)kvh * a.kA_hs;
     const bf16* kB = DB ? a.kB + (size_t)slot * a.kB_ss : nullptr;
     const bf16* vb = a.v + (size_t)slot * a.v_ss + (size_t)kvh * a.v_hs + (size_t)blockIdx.z * DV;
@@ -1043,7 +1046,7 @@ __global__ void __launch_bounds__(128, 2) window_attn_mma_kernel(const WinMma a)
       for (int nt = 0; nt < 2; ++nt) {
         const int jj = kb + 8 * nt + gid;
         const bool ok = jj < nkeys;
-        const int row = ok ? (jlo + jj) % a.cap : 0;
+        const int row = ok ? key_row(jj) : 0;
         const bf16* kp = kA + (size_t)row * a.kA_rs;
 #pragma unroll
         for (int j = 0; j < DA / 32; ++j) r.k[nt][j] = ok ? __ldg(reinterpret_cast<const uint4*>(kp + 32 * j + 8 * tig)) : zero4;
@@ -1057,7 +1060,7 @@ __global__ void __launch_bounds__(128, 2) window_attn_mma_kernel(const WinMma a)
       for (int q = 0; q < 4; ++q) {
         const int jj = kb + 2 * tig + (q & 1) + 8 * (q >> 1);
         const bool ok = jj < nkeys;
-        const bf16* vp = vb + (size_t)(ok ? (jlo + jj) % a.cap : 0) * a.v_rs;
+        const bf16* vp = vb + (size_t)(ok ? key_row(jj) : 0) * a.v_rs;
 #pragma unroll
         for (int sp = 0; sp < DV / 64; ++sp) r.v[q][sp] = ok ? __ldg(reinterpret_cast<const uint4*>(vp + 64 * sp + 8 * gid)) : zero4;
       }
@@ -1081,7 +1084,7 @@ __global__ void __launch_bounds__(128, 2) window_attn_mma_kernel(const WinMma a)
         for (int nt = 0; nt < 2; ++nt) {
           const int jj = kb + 8 * nt + gid;
           okk[nt] = jj < nkeys;
-          const int row = okk[nt] ? (jlo + jj) % a.cap : 0;
+          const int row = okk[nt] ? key_row(jj) : 0;
           kp[nt] = kA + (size_t)row * a.kA_rs + 8 * tig;
           kq[nt] = DB ? kB + (size_t)row * a.kB_rs + 8 * tig : nullptr;
         }
@@ -1103,7 +1106,7 @@ __global__ void __launch_bounds__(128, 2) window_attn_mma_kernel(const WinMma a)
         for (int q = 0; q < 4; ++q) {                       // this step's value rows, in flight during the softmax
           const int jj = kb + 2 * tig + (q & 1) + 8 * (q >> 1);
           const bool ok = jj < nkeys;
-          const bf16* vp = vb + (size_t)(ok ? (jlo + jj) % a.cap : 0) * a.v_rs;
+          const bf16* vp = vb + (size_t)(ok ? key_row(jj) : 0) * a.v_rs;
 #pragma unroll
           for (int sp = 0; sp < DV / 64; ++sp) cur.v[q][sp] = ok ? __ldg(reinterpret_cast<const uint4*>(vp + 64 * sp + 8 * gid)) : zero4;
         }
@@ -1125,9 +1128,9 @@ __global__ void __launch_bounds__(128, 2) window_attn_mma_kernel(const WinMma a)
       for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
         for (int c = 0; c < 4; ++c) {
-          const int pj = jlo + kb + 8 * nt + 2 * tig + (c & 1);
+          const int jj = kb + 8 * nt + 2 * tig + (c & 1), pj = jj < nk ? jj : jlo + jj - nk;
           const int pr = (c >> 1) ? posB : posA;
-          const bool vis = ((c >> 1) ? inB : inA) && pj <= pr && pr - pj < a.window && pj <= pmax;
+          const bool vis = ((c >> 1) ? inB : inA) && pj <= pr && (pr - pj < a.window || pj < a.keep) && jj < nkeys;
           s[nt][c] = vis ? s[nt][c] * a.scale : -INFINITY;
           if (c >> 1) mxB = fmaxf(mxB, s[nt][c]); else mxA = fmaxf(mxA, s[nt][c]);
         }
@@ -1198,9 +1201,9 @@ __global__ void __launch_bounds__(128, 2) window_attn_mma_kernel(const WinMma a)
       L += sL[w][row] * f;
       acc += sO[(w * 16 + row) * DV + d] * f;
     }
-    float r = acc / L;
+    float r = acc / L * a.out_scale;
     if (a.gate) r *= __fdividef(1.0f, 1.0f + __expf(-__bfloat162float(a.gate[(size_t)tok * a.gate_ld + (a.gate_per_head ? (size_t)head : (size_t)head * a.out_hs + (size_t)blockIdx.z * DV + d)])));
-    a.out[((size_t)tok * a.H + head) * a.out_hs + (size_t)blockIdx.z * DV + d] = __float2bfloat16_rn(r);
+    a.out[(size_t)tok * a.out_ts + (size_t)head * a.out_hs + (size_t)blockIdx.z * DV + d] = __float2bfloat16_rn(r);
   }
 }
 
@@ -1468,16 +1471,18 @@ __global__ void __launch_bounds__(32 * NW, NW == 4 ? 2 : 1) prompt_attn_mma_kern
   }
   const int last = pos0 + min(i0 + BM, a.ntok) - 1;                     // last key any row of the block sees
   const int start = max(0, pos0 + i0 - a.window + 1);                    // first key the block's first row sees
-  const int ntiles = (last - start + BN) / BN;
+  // keys in order: nk kept positions that the first row's window has left behind, then positions from `start` on
+  const int nk = min(a.keep, start), nkeys = nk + last - start + 1;
+  const int ntiles = (nkeys + BN - 1) / BN;
   const bf16* kA = a.kA + (size_t)slot * a.kA_ss + (size_t)kvh * a.kA_hs;
   const bf16* kB = DB ? a.kB + (size_t)slot * a.kB_ss : nullptr;
   const bf16* vb = a.v + (size_t)slot * a.v_ss + (size_t)kvh * a.v_hs;
   // TPK threads per key row: one row index (position % cap) per thread and tile, then straight runs of 16-byte pieces
   const int lkey = tid / TPK, lhalf = tid % TPK;
   auto load_tile = [&](int t, int buf) {
-    const int j = start + t * BN + lkey;
-    const bool ok = j <= last;
-    const int row = ok ? j % a.cap : 0;
+    const int jj = t * BN + lkey;
+    const bool ok = jj < nkeys;
+    const int row = ok ? ring_row(jj < nk ? jj : start + jj - nk, a.keep, a.cap) : 0;
     bf16* dK = sK + ((size_t)buf * BN + lkey) * KS;
     bf16* dV = sV + ((size_t)buf * BN + lkey) * VS;
     const bf16* srcA = kA + (size_t)row * a.kA_rs;
@@ -1524,7 +1529,7 @@ __global__ void __launch_bounds__(32 * NW, NW == 4 ? 2 : 1) prompt_attn_mma_kern
       asm volatile("cp.async.wait_group 0;\n" ::: "memory");
     }
     __syncthreads();
-    const int j0 = start + t * BN;
+    const int jt = t * BN, j0 = jt < nk ? jt : start + jt - nk;          // the tile's first position (positions ascend)
     if (j0 <= wlast) {                                                   // a tile past this warp's rows holds nothing for it
       const bf16* K = sK + (size_t)buf * BN * KS;
       const bf16* V = sV + (size_t)buf * BN * VS;
@@ -1543,7 +1548,7 @@ __global__ void __launch_bounds__(32 * NW, NW == 4 ? 2 : 1) prompt_attn_mma_kern
       float mxA = -INFINITY, mxB = -INFINITY;
       // a tile that lies wholly before the warp's first row and inside its last row's window needs no mask (most tiles)
       const int wfirst = pos0 + i0 + warp * 16;
-      if (j0 + BN - 1 <= wfirst && j0 + BN - 1 <= last && (wfirst + 15) - j0 < a.window) {
+      if (jt >= nk && j0 + BN - 1 <= wfirst && j0 + BN - 1 <= last && (wfirst + 15) - j0 < a.window) {
 #pragma unroll
         for (int nt = 0; nt < BN / 8; ++nt) {
 #pragma unroll
@@ -1556,9 +1561,9 @@ __global__ void __launch_bounds__(32 * NW, NW == 4 ? 2 : 1) prompt_attn_mma_kern
         for (int nt = 0; nt < BN / 8; ++nt)
 #pragma unroll
           for (int c = 0; c < 4; ++c) {
-            const int pj = j0 + nt * 8 + 2 * tig + (c & 1);
+            const int jj = jt + nt * 8 + 2 * tig + (c & 1), pj = jj < nk ? jj : start + jj - nk;
             const int pr = (c >> 1) ? posB : posA;
-            const bool vis = pj <= pr && pr - pj < a.window && pj <= last;
+            const bool vis = pj <= pr && (pr - pj < a.window || pj < a.keep) && jj < nkeys;
             s[nt][c] = vis ? s[nt][c] * a.scale : -INFINITY;
             if (c >> 1) mxB = fmaxf(mxB, s[nt][c]); else mxA = fmaxf(mxA, s[nt][c]);
           }
@@ -1616,10 +1621,10 @@ __global__ void __launch_bounds__(32 * NW, NW == 4 ? 2 : 1) prompt_attn_mma_kern
       f = m == -INFINITY ? 0.f : __expf(m - M);
       L = l * f + __expf(a.sink[head] - M);
     }
-    float inv = L > 0.f ? f / L : 0.f;
+    float inv = L > 0.f ? f / L * a.out_scale : 0.f;
     const bf16* gp = a.gate ? a.gate + (size_t)tok * a.gate_ld + (a.gate_per_head ? (size_t)head : (size_t)head * DV) : nullptr;
     if (gp && a.gate_per_head) inv *= __fdividef(1.0f, 1.0f + __expf(-__bfloat162float(gp[0])));
-    bf16* orow = a.out + ((size_t)tok * a.H + head) * DV;
+    bf16* orow = a.out + (size_t)tok * a.out_ts + (size_t)head * DV;
 #pragma unroll
     for (int nt = 0; nt < DV / 8; ++nt) {
       const int d = nt * 8 + 2 * tig;
@@ -1665,7 +1670,7 @@ bool prompt_mma_shape(int DA, int DB, int DV) {
 int prompt_attention_mma(const qspec_window_attn_args* p, const void* kB, long long kB_ss, int kB_rs, int DB, int slot, int pos0,
                          cudaStream_t st) {
   const int DA = p->DA, DV = p->DV;
-  const bool ok = prompt_mma_shape(DA, DB, DV) && p->H % p->G == 0 && p->H <= 65535 && p->k_row_stride % 8 == 0 && p->k_head_stride % 8 == 0 &&
+  const bool ok = prompt_mma_shape(DA, DB, DV) && p->keep_first >= 0 && p->keep_first < p->cap && p->out_tok_stride % 2 == 0 && p->H % p->G == 0 && p->H <= 65535 && p->k_row_stride % 8 == 0 && p->k_head_stride % 8 == 0 &&
                   p->k_slot_stride % 8 == 0 && p->v_row_stride % 8 == 0 && p->v_head_stride % 8 == 0 && p->v_slot_stride % 8 == 0 &&
                   kB_rs % 8 == 0 && kB_ss % 8 == 0 && p->qa_tok_stride % 2 == 0 && p->qa_head_stride % 2 == 0 &&
                   (((uintptr_t)p->k | (uintptr_t)p->v | (uintptr_t)kB) & 15) == 0 && ((uintptr_t)p->qa & 7) == 0 && ((uintptr_t)p->out & 3) == 0;
@@ -1678,6 +1683,8 @@ int prompt_attention_mma(const qspec_window_attn_args* p, const void* kB, long l
   a.sink = p->sink; a.gate = (const bf16*)p->gate; a.gate_ld = p->gate_ld; a.gate_per_head = p->gate_per_head;
   a.out = (bf16*)p->out; a.out_hs = DV; a.meta = p->meta; a.ntok = p->ntok; a.H = p->H; a.G = p->G; a.window = p->window; a.cap = p->cap;
   a.scale = p->scale; a.token_rows = 1;
+  a.keep = p->keep_first; a.out_ts = p->out_tok_stride ? p->out_tok_stride : (long long)p->H * DV;
+  a.out_scale = p->out_scale != 0.f ? p->out_scale : 1.0f;
   if (DB) return launch_prompt_attn<128, 64, 128>(a, slot, pos0, st);
   if (DA == 128) return launch_prompt_attn<128, 0, 128>(a, slot, pos0, st);
   return launch_prompt_attn<64, 0, 64>(a, slot, pos0, st);
@@ -1711,7 +1718,7 @@ bool window_mma_shape(int DA, int DB, int DV) {
 int window_attention_mma(const qspec_window_attn_args* p, const void* kB, long long kB_ss, int kB_rs, int DB, int token_rows,
                          cudaStream_t st) {
   const int DA = p->DA, DV = p->DV;
-  const bool ok = window_mma_shape(DA, DB, DV) && p->H % p->G == 0 && (token_rows || p->H / p->G <= 16) && p->H <= 65535 && p->G <= 65535 &&
+  const bool ok = window_mma_shape(DA, DB, DV) && p->keep_first >= 0 && p->keep_first < p->cap && p->H % p->G == 0 && (token_rows || p->H / p->G <= 16) && p->H <= 65535 && p->G <= 65535 &&
                   p->k_row_stride % 8 == 0 && p->k_head_stride % 8 == 0 && p->k_slot_stride % 8 == 0 && p->v_row_stride % 8 == 0 &&
                   p->v_head_stride % 8 == 0 && p->v_slot_stride % 8 == 0 && kB_rs % 8 == 0 && kB_ss % 8 == 0 &&
                   p->qa_tok_stride % 2 == 0 && p->qa_head_stride % 2 == 0 &&
@@ -1725,10 +1732,13 @@ int window_attention_mma(const qspec_window_attn_args* p, const void* kB, long l
   a.sink = p->sink; a.gate = (const bf16*)p->gate; a.gate_ld = p->gate_ld; a.gate_per_head = p->gate_per_head;
   a.out = (bf16*)p->out; a.out_hs = DV; a.meta = p->meta; a.ntok = p->ntok; a.H = p->H; a.G = p->G; a.window = p->window; a.cap = p->cap;
   a.scale = p->scale; a.token_rows = token_rows;
+  a.keep = p->keep_first; a.out_ts = p->out_tok_stride ? p->out_tok_stride : (long long)p->H * DV;
+  a.out_scale = p->out_scale != 0.f ? p->out_scale : 1.0f;
   // a latent cache read in the absorbed form (keys and values are the same rows): the CTA-level kernel; QSPEC_SEQ_LATENT=sliced
   // keeps the form with one CTA per slice of 128 value columns, for comparison
   static const bool sliced = [] { const char* v = getenv("QSPEC_SEQ_LATENT"); return v && !strcmp(v, "sliced"); }();
-  if (!sliced && !token_rows && DA >= 256 && DV == DA && p->v == p->k && (!p->gate || p->gate_per_head)) {
+  const bool plain_rows = p->keep_first == 0 && !p->out_tok_stride && a.out_scale == 1.0f;
+  if (!sliced && plain_rows && !token_rows && DA >= 256 && DV == DA && p->v == p->k && (!p->gate || p->gate_per_head)) {
     if (DA == 512) return launch_latent_absorbed<512>(a, st);
     return launch_latent_absorbed<256>(a, st);
   }

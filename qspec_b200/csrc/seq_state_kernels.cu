@@ -9,18 +9,6 @@
 
 namespace qspec {
 
-// 4-byte asynchronous copies into shared memory (both addresses on 4-byte boundaries)
-__device__ __forceinline__ void cp_async_4(float* smem_dst, const float* src) {
-  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;\n" ::"r"((uint32_t)__cvta_generic_to_shared(smem_dst)), "l"(src) : "memory");
-}
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;\n" ::: "memory"); }
-template <int N> __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;\n" ::"n"(N) : "memory"); }
-
-// 16-byte asynchronous copy into shared memory; `valid` false writes zeros and reads nothing
-__device__ __forceinline__ void cp_async_16z(void* smem_dst, const void* src, bool valid) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"((uint32_t)__cvta_generic_to_shared(smem_dst)), "l"(src),
-               "r"(valid ? 16 : 0) : "memory");
-}
 __device__ __forceinline__ void tk_ldmatrix_x4(uint32_t (&r)[4], const __nv_bfloat16* p) {
   const uint32_t a = (uint32_t)__cvta_generic_to_shared(p);
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];\n" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
@@ -43,9 +31,6 @@ __device__ __forceinline__ void tk_mma_16816(float (&c)[4], const uint32_t (&a)[
                : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
                : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
-
-__device__ __forceinline__ float silu_f(float z) { return z / (1.0f + expf(-z)); }
-__device__ __forceinline__ float softplus_f(float z) { return z > 20.f ? z : log1pf(expf(z)); }
 
 // ---- short causal convolution over time, per channel, with an activation ---------------------------------------------------
 // out[t, c] = act(bias[c] + sum_j w[c, j] * in[t - taps + 1 + j, c]). Rows before the segment's first token come from the

@@ -1010,20 +1010,28 @@ def seq_qkv_prep(p: torch.Tensor, HD: int, GD: int, GDV: int, qn_w: torch.Tensor
          "seq_qkv_prep")
 
 
+def _att_out(t: torch.Tensor, name: str, dtypes) -> None:
+    """An attention output [ntok, H, DV]: contiguous heads of a token, any token stride (a column range of a wider buffer)."""
+    if t is None or not t.is_cuda or t.dim() != 3 or t.dtype not in dtypes or t.stride(2) != 1 or (t.shape[1] > 1 and t.stride(1) != t.shape[2]):
+        raise ValueError(f"{name}: a CUDA tensor [ntok, H, DV] of {dtypes} with contiguous heads expected")
+
+
 def seq_window_attention(qa: torch.Tensor, qb: Optional[torch.Tensor], cache_k: torch.Tensor, cache_v: torch.Tensor, out: torch.Tensor,
                          meta: torch.Tensor, window: int, scale: float, sink: Optional[torch.Tensor] = None,
-                         gate: Optional[torch.Tensor] = None, gate_per_head: bool = False) -> None:
+                         gate: Optional[torch.Tensor] = None, gate_per_head: bool = False, keep_first: int = 0, out_scale: float = 1.0) -> None:
     """Sliding-window softmax attention with a per-head sink over ring caches.
     qa [ntok, H, DA] and qb [ntok, H, DB] (float32, any strides with a unit last stride): the two parts of the query;
     cache_k [slots, cap, G, DA + DB], cache_v [slots, cap, G, DV] (views with a unit last stride: a latent cache passes two
     views of one buffer); out [ntok, H, DV]; gate [ntok, >= H * DV] (sigmoid applied) or None; gate_per_head: gate is [ntok, >= H],
-    one number per head. sink None: an ordinary softmax."""
+    one number per head. sink None: an ordinary softmax. keep_first: the first positions every later token keeps seeing, in ring rows
+    that are never reused (cache rows as `seq_head_prep` writes them). out: rows of H * DV contiguous elements, any token stride;
+    multiplied by out_scale."""
     import ctypes
     if qa.dtype != _F32 or (qb is not None and qb.dtype != _F32):
         raise ValueError("seq_window_attention: queries are float32")
     if cache_k.dtype != out.dtype or cache_v.dtype != out.dtype or (gate is not None and gate.dtype != out.dtype):
         raise ValueError("seq_window_attention: caches, gate and out share one element type")
-    _chk(out, "out", _SEQ_ACT)
+    _att_out(out, "out", _SEQ_ACT)
     ntok, H, DA = qa.shape
     DB = qb.shape[2] if qb is not None else 0
     slots, cap, G, DK = cache_k.shape
@@ -1039,7 +1047,8 @@ def seq_window_attention(qa: torch.Tensor, qb: Optional[torch.Tensor], cache_k: 
                             cache_k.data_ptr(), cache_k.stride(0), cache_k.stride(1), cache_k.stride(2),
                             cache_v.data_ptr(), cache_v.stride(0), cache_v.stride(1), cache_v.stride(2), DV,
                             _ptr(sink), gate.data_ptr() if gate is not None else None, gate.stride(0) if gate is not None else 0,
-                            _ptr(out), _ptr(meta), ntok, H, G, int(window), cap, float(scale), int(gate_per_head))
+                            out.data_ptr(), _ptr(meta), ntok, H, G, int(window), cap, float(scale), int(gate_per_head), int(keep_first),
+                            out.stride(0), float(out_scale))
     _seq(_lib.load_seq().qspec_seq_window_attention(ctypes.byref(a), _sdt(out), _stream()), "seq_window_attention")
 
 
@@ -1052,7 +1061,7 @@ def seq_window_attention_mma_supported(out_dtype, DA: int, DB: int, DV: int, H: 
 def seq_window_attention_mma(q: torch.Tensor, cache_k: torch.Tensor, k_shared: Optional[torch.Tensor], cache_v: torch.Tensor,
                              out: torch.Tensor, meta: torch.Tensor, window: int, scale: float, token_rows: bool,
                              sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
-                             gate_per_head: bool = False) -> None:
+                             gate_per_head: bool = False, keep_first: int = 0, out_scale: float = 1.0) -> None:
     """`seq_window_attention` on the tensor cores (bfloat16). q [ntok, H, DK] float32; cache_k [slots, cap, G, DA] holds the
     per-head part of the keys and k_shared [slots, cap, DB] (or None) the part all heads share, DK = DA + DB; cache_v
     [slots, cap, G, DV] (views: a slot stride of 0 serves one buffer to every slot). token_rows: False = the rows of the
@@ -1061,7 +1070,7 @@ def seq_window_attention_mma(q: torch.Tensor, cache_k: torch.Tensor, k_shared: O
     import ctypes
     if q.dtype != _F32 or cache_k.dtype != _BF16 or cache_v.dtype != _BF16 or out.dtype != _BF16:
         raise ValueError("seq_window_attention_mma: float32 queries, bfloat16 caches and output")
-    _chk(out, "out", (_BF16,))
+    _att_out(out, "out", (_BF16,))
     ntok, H, DK = q.shape
     slots, cap, G, DA = cache_k.shape
     DB = k_shared.shape[2] if k_shared is not None else 0
@@ -1076,7 +1085,8 @@ def seq_window_attention_mma(q: torch.Tensor, cache_k: torch.Tensor, k_shared: O
                             cache_k.data_ptr(), cache_k.stride(0), cache_k.stride(1), cache_k.stride(2),
                             cache_v.data_ptr(), cache_v.stride(0), cache_v.stride(1), cache_v.stride(2), DV,
                             _ptr(sink), gate.data_ptr() if gate is not None else None, gate.stride(0) if gate is not None else 0,
-                            _ptr(out), _ptr(meta), ntok, H, G, int(window), cap, float(scale), int(gate_per_head))
+                            out.data_ptr(), _ptr(meta), ntok, H, G, int(window), cap, float(scale), int(gate_per_head), int(keep_first),
+                            out.stride(0), float(out_scale))
     _seq(_lib.load_seq().qspec_seq_window_attention_mma(ctypes.byref(a), k_shared.data_ptr() if k_shared is not None else None,
                                                         k_shared.stride(0) if k_shared is not None else 0,
                                                         k_shared.stride(1) if k_shared is not None else 0, DB, int(token_rows), _stream()),
@@ -1188,10 +1198,11 @@ def seq_lightning(p: torch.Tensor, decay: torch.Tensor, norm_w: torch.Tensor, st
 
 def moe_route_grouped(h: torch.Tensor, router_w: torch.Tensor, correction: Optional[torch.Tensor], idx: torch.Tensor,
                       weight: torch.Tensor, *, score: str = "sigmoid", groups: int = 1, keep: int = 1, group_top: int = 2,
-                      scale: float = 1.0, extra: Optional[torch.Tensor] = None) -> None:
+                      scale: float = 1.0, normalize: bool = False, extra: Optional[torch.Tensor] = None) -> None:
     """Router with expert groups: scores s = sigmoid or softmax of router_w h (float32), choice = s + correction; the experts form
     `groups` equal groups of neighbours, a group scores the sum of its `group_top` largest choices and only the `keep` best groups
-    stay; idx int32 [ntok, top] = the largest remaining choices, weight float32 [ntok, top] = scale * s. Rows of router_w past the
+    stay; idx int32 [ntok, top] = the largest remaining choices, weight float32 [ntok, top] = scale * s, divided by the sum of the
+    chosen s (+ 1e-20) if normalize. Rows of router_w past the
     experts ([R + n, W]) are gate rows: extra float32 [ntok, n] (a view with a unit last stride) receives their sigmoid."""
     _chk(h, "h", _SEQ_ACT); _chk(router_w, "router_w", (_F32,)); _chk(correction, "correction", (_F32,), allow_none=True)
     _chk(idx, "idx", (torch.int32,)); _chk(weight, "weight", (_F32,))
@@ -1210,7 +1221,7 @@ def moe_route_grouped(h: torch.Tensor, router_w: torch.Tensor, correction: Optio
                                                  extra.data_ptr() if extra is not None else None,
                                                  extra.stride(0) if extra is not None else 0, ntok, W, R, top,
                                                  {"softmax": 0, "sigmoid": 1}[score], int(groups), int(keep), int(group_top),
-                                                 float(scale), n_extra, _sdt(h), _stream()), "moe_route_grouped")
+                                                 float(scale), int(normalize), n_extra, _sdt(h), _stream()), "moe_route_grouped")
 
 
 def seq_prompt_attention_mma_supported(out_dtype, DA: int, DB: int, DV: int) -> bool:
@@ -1222,7 +1233,7 @@ def seq_prompt_attention_mma_supported(out_dtype, DA: int, DB: int, DV: int) -> 
 def seq_prompt_attention_mma(q: torch.Tensor, cache_k: torch.Tensor, k_shared: Optional[torch.Tensor], cache_v: torch.Tensor,
                              out: torch.Tensor, slot: int, pos0: int, window: int, scale: float,
                              sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
-                             gate_per_head: bool = False) -> None:
+                             gate_per_head: bool = False, keep_first: int = 0, out_scale: float = 1.0) -> None:
     """Softmax attention of one prompt portion on the tensor cores (bfloat16): the rows of q [ntok, H, DK] (float32) are the
     consecutive positions pos0 .. pos0 + ntok - 1 of the sequence in `slot`. 64 tokens and one head per CTA; every visible key /
     value row is read once per 64 queries. cache_k [slots, cap, G, DA], k_shared [slots, cap, DB] or None (DK = DA + DB), cache_v
@@ -1230,7 +1241,7 @@ def seq_prompt_attention_mma(q: torch.Tensor, cache_k: torch.Tensor, k_shared: O
     import ctypes
     if q.dtype != _F32 or cache_k.dtype != _BF16 or cache_v.dtype != _BF16 or out.dtype != _BF16:
         raise ValueError("seq_prompt_attention_mma: float32 queries, bfloat16 caches and output")
-    _chk(out, "out", (_BF16,))
+    _att_out(out, "out", (_BF16,))
     ntok, H, DK = q.shape
     slots, cap, G, DA = cache_k.shape
     DB = k_shared.shape[2] if k_shared is not None else 0
@@ -1245,7 +1256,8 @@ def seq_prompt_attention_mma(q: torch.Tensor, cache_k: torch.Tensor, k_shared: O
                             cache_k.data_ptr(), cache_k.stride(0), cache_k.stride(1), cache_k.stride(2),
                             cache_v.data_ptr(), cache_v.stride(0), cache_v.stride(1), cache_v.stride(2), DV,
                             _ptr(sink), gate.data_ptr() if gate is not None else None, gate.stride(0) if gate is not None else 0,
-                            _ptr(out), None, ntok, H, G, int(window), cap, float(scale), int(gate_per_head))
+                            out.data_ptr(), None, ntok, H, G, int(window), cap, float(scale), int(gate_per_head), int(keep_first),
+                            out.stride(0), float(out_scale))
     _seq(_lib.load_seq().qspec_seq_prompt_attention_mma(ctypes.byref(a), k_shared.data_ptr() if k_shared is not None else None,
                                                         k_shared.stride(0) if k_shared is not None else 0,
                                                         k_shared.stride(1) if k_shared is not None else 0, DB, int(slot), int(pos0),
@@ -1396,3 +1408,110 @@ def seq_scale(a: torch.Tensor, s: float) -> None:
     """a <- s * a in place (float32)."""
     _chk(a, "a", (_F32,))
     _seq(_lib.load_seq().qspec_seq_scale_f32(_ptr(a), a.numel(), float(s), _stream()), "seq_scale")
+
+
+# ---- norm without statistics, heads prepared from the projection, delta rule with channel decays, logit soft cap ------------------
+def seq_residual_tanh(x_in: torch.Tensor, alpha: float, w: Optional[torch.Tensor], b: Optional[torch.Tensor], *,
+                      y: Optional[torch.Tensor] = None, y_w: Optional[torch.Tensor] = None, y_bias: Optional[torch.Tensor] = None,
+                      mult: float = 1.0, x_out: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None) -> None:
+    """r = x_in + mult * (sum of y's parts, each times y_w [ntok, parts] if given, + y_bias); out = tanh(alpha * r) * w + b. y [ntok, W]
+    or [ntok, parts, W]; y_bias float32 [W] or None; r goes to x_out (float32; may be x_in), the norm to out (activation type)."""
+    _chk(x_in, "x_in", (_F32,)); _chk(x_out, "x_out", (_F32,), allow_none=True); _chk(out, "out", _SEQ_ACT, allow_none=True)
+    _chk(w, "w", (_F32,), allow_none=out is None); _chk(b, "b", (_F32,), allow_none=out is None)
+    _chk(y, "y", _SEQ_ACT, allow_none=True); _chk(y_w, "y_w", (_F32,), allow_none=True); _chk(y_bias, "y_bias", (_F32,), allow_none=True)
+    ntok, W = x_in.shape
+    parts, pstride, tstride = 1, 0, W
+    if y is not None:
+        if y.dim() == 3:
+            parts, pstride, tstride = y.shape[1], W, y.shape[1] * W
+        if y.shape[0] != ntok or y.shape[-1] != W or (y_w is not None and y_w.shape != (ntok, parts)):
+            raise ValueError("seq_residual_tanh: y / y_w shapes do not match x")
+    if any(t is not None and t.shape != (ntok, W) for t in (x_out, out)) or any(t is not None and t.numel() != W for t in (w, b, y_bias)):
+        raise ValueError("seq_residual_tanh: shapes do not match")
+    act = _sdt(out) if out is not None else (_sdt(y) if y is not None else _lib.DTYPE_F32)
+    _seq(_lib.load_seq().qspec_seq_residual_tanh(_ptr(x_in), _ptr(x_out), _ptr(y), parts, pstride, tstride, _ptr(y_w), _ptr(y_bias),
+                                                 float(mult), float(alpha), _ptr(w), _ptr(b), _ptr(out), ntok, W,
+                                                 _sdt(y) if y is not None else act, act, _stream()), "seq_residual_tanh")
+
+
+def seq_softcap(a: torch.Tensor, cap: float) -> None:
+    """a <- cap * tanh(a / cap) in place (float32)."""
+    _chk(a, "a", (_F32,))
+    _seq(_lib.load_seq().qspec_seq_softcap_f32(_ptr(a), a.numel(), float(cap), _stream()), "seq_softcap")
+
+
+def seq_head_prep(p: torch.Tensor, q_off: int, k_off: int, v_off: Optional[int], qout: torch.Tensor, cache_k: torch.Tensor,
+                  cache_v: torch.Tensor, meta: torch.Tensor, H: int, eps: float, *, conv_w: Optional[torch.Tensor] = None,
+                  tail: Optional[torch.Tensor] = None, qn_w: Optional[torch.Tensor] = None, kn_w: Optional[torch.Tensor] = None,
+                  norm_last: bool = False, inv_freq: Optional[torch.Tensor] = None, rot_dims: int = 0, rot_amp: float = 1.0,
+                  temp_coef: float = 0.0, temp_every: int = 0, keep_first: int = 0) -> None:
+    """Attention heads from the projection rows p [ntok, ld] (q [H x D], k [G x D], v [G x DV] at the given columns; v_off None: the
+    values are the keys as projected): short convolution over q, k, v (conv_w float32 [taps, H D + G D + G DV], the last row meets the
+    current token; tail float32 [2, slots, taps - 1, channels]), unit-RMS norm per head with the weights qn_w / kn_w (None: ones) before
+    the rotation -- after it if norm_last --, rotation of the first rot_dims entries by pos * inv_freq with the amplitude rot_amp, and
+    q * (1 + temp_coef ln(floor((pos + 1) / temp_every) + 1)) if temp_every > 0. qout float32 [ntok, H, D]; cache_k [slots, cap, G, D]
+    and cache_v [slots, cap, G, DV] of p's type take ring row pos, the first keep_first rows never reused."""
+    import ctypes
+    _rows(p, "p", _SEQ_ACT); _chk(qout, "qout", (_F32,)); _chk(cache_k, "cache_k", (p.dtype,)); _chk(cache_v, "cache_v", (p.dtype,))
+    for t, n in ((conv_w, "conv_w"), (qn_w, "qn_w"), (kn_w, "kn_w"), (inv_freq, "inv_freq")):
+        _chk(t, n, (_F32,), allow_none=True)
+    ntok = p.shape[0]
+    slots, cap, G, D = cache_k.shape
+    DV = cache_v.shape[3]
+    C = H * D + G * D + G * DV
+    taps = conv_w.shape[0] if conv_w is not None else 0
+    if cache_v.shape[:3] != (slots, cap, G) or qout.shape != (ntok, H, D) or meta.shape != (5, ntok) or \
+            any(t is not None and t.numel() != D for t in (qn_w, kn_w)) or (rot_dims and (inv_freq is None or inv_freq.numel() != rot_dims // 2)):
+        raise ValueError("seq_head_prep: shapes do not match")
+    if conv_w is not None:
+        _chk(tail, "tail", (_F32,))
+        if conv_w.shape != (taps, C) or tail.shape != (2, slots, taps - 1, C):
+            raise ValueError("seq_head_prep: the convolution and its tail have H D + G D + G DV channels")
+    a = _lib.HeadPrepArgs(p.data_ptr(), p.stride(0), int(q_off), int(k_off), -1 if v_off is None else int(v_off), _ptr(conv_w), taps,
+                          _ptr(tail), slots, _ptr(qn_w), _ptr(kn_w), int(norm_last), _ptr(inv_freq), int(rot_dims), float(rot_amp),
+                          float(temp_coef), int(temp_every), _ptr(qout), _ptr(cache_k), _ptr(cache_v), cap, int(keep_first), _ptr(meta),
+                          ntok, H, G, D, DV, float(eps))
+    _seq(_lib.load_seq().qspec_seq_head_prep(ctypes.byref(a), _sdt(p), _stream()), "seq_head_prep")
+
+
+def seq_delta_channel_scratch_bytes(nblocks: int, ntok: int, H: int, D: int, DV: int) -> int:
+    """Bytes of scratch that `seq_delta_channel` needs for nblocks blocks of 16 tokens in a step of ntok tokens."""
+    return int(_lib.load_seq().qspec_seq_delta_channel_scratch_bytes(int(nblocks), int(ntok), H, D, DV))
+
+
+def seq_delta_channel(p: torch.Tensor, beta_off: int, conv_w: torch.Tensor, tail: torch.Tensor, decay: torch.Tensor, A_log: torch.Tensor,
+                      dt_bias: torch.Tensor, norm_w: torch.Tensor, gate: Optional[torch.Tensor], state: torch.Tensor, out: torch.Tensor,
+                      meta, G: int, eps: float, *, scratch: Optional[torch.Tensor] = None, unit_eps: float = 1e-6,
+                      q_mult: Optional[float] = None, out_scale: float = 1.0) -> None:
+    """Gated delta rule with one decay per head and key channel, from the projection rows p = [q (G x D) | k (G x D) | v (H x DV) | ...,
+    H step-size logits at column beta_off] to the gated output: convolution (conv_w float32 [taps, channels]) and silu, unit q and k, g =
+    exp(-exp(A_log) softplus(decay + dt_bias)) with decay float32 [ntok, H * D]; per head S <- diag(g) S; u = sigmoid(beta) (v - S^T k);
+    S <- S + k u^T; o = S^T q; out [ntok, H * DV] (view) = out_scale * unit_rms(o) * norm_w * sigmoid(gate). state float32 [slots, H, D,
+    DV]. meta: the step's `state.BatchMeta`; its segments longer than SCAN_SHORT tokens take the block form, which needs scratch (uint8)."""
+    import ctypes
+    from .state import SCAN_SHORT
+    _rows(p, "p", _SEQ_ACT); _rows(decay, "decay", (_F32,)); _rows(out, "out", (p.dtype,)); _chk(state, "state", (_F32,))
+    for t, n in ((conv_w, "conv_w"), (tail, "tail"), (A_log, "A_log"), (dt_bias, "dt_bias"), (norm_w, "norm_w")):
+        _chk(t, n, (_F32,))
+    if gate is not None:
+        _rows(gate, "gate", (p.dtype,))
+    ntok = p.shape[0]
+    slots, H, D, DV = state.shape
+    C = 2 * G * D + H * DV
+    taps = conv_w.shape[0]
+    if conv_w.shape != (taps, C) or tail.shape != (2, slots, taps - 1, C) or p.shape[1] < C or not 0 <= beta_off <= p.shape[1] - H or \
+            decay.shape != (ntok, H * D) or out.shape != (ntok, H * DV) or A_log.numel() != H or dt_bias.numel() != H * D or \
+            norm_w.numel() != DV or meta.table.shape != (5, ntok) or (gate is not None and gate.shape != (ntok, H * DV)):
+        raise ValueError("seq_delta_channel: shapes do not match")
+    a = _lib.DeltaChannelArgs(p.data_ptr(), p.stride(0), int(beta_off), _ptr(conv_w), taps, _ptr(tail), slots, decay.data_ptr(),
+                              decay.stride(0), _ptr(A_log), _ptr(dt_bias), _ptr(norm_w), gate.data_ptr() if gate is not None else None,
+                              gate.stride(0) if gate is not None else 0, _ptr(state), out.data_ptr(), out.stride(0), _ptr(meta.table),
+                              _ptr(meta.seg_starts), meta.seg_starts.numel(), ntok, H, G, D, DV, float(unit_eps),
+                              float(D ** -0.5 if q_mult is None else q_mult), float(eps), float(out_scale))
+    nlong, nblk = meta.long_starts.numel(), meta.block_rows.numel()
+    _seq(_lib.load_seq().qspec_seq_delta_channel(ctypes.byref(a), meta.block_rows.data_ptr() if nlong else None, nblk,
+                                                 meta.long_starts.data_ptr() if nlong else None,
+                                                 meta.long_block0.data_ptr() if nlong else None, nlong, SCAN_SHORT,
+                                                 scratch.data_ptr() if scratch is not None else None,
+                                                 scratch.numel() * scratch.element_size() if scratch is not None else 0, _sdt(p), _stream()),
+         "seq_delta_channel")
