@@ -82,6 +82,10 @@ __device__ __forceinline__ void pdl_enter() {
 #endif
 }
 
+// For kernels of several waves of CTAs whose dependent would take SM resources from them while it waits: the dependent starts when
+// this grid has finished.
+__device__ __forceinline__ void pdl_enter_hold() { asm volatile("griddepcontrol.wait;\n" ::: "memory"); }
+
 // ---- thread-block clusters: distributed shared memory ----------------------------------------
 __device__ __forceinline__ uint32_t mapa_shared(uint32_t addr, uint32_t rank) {
   uint32_t r;

@@ -372,9 +372,9 @@ constexpr int DBLK = 16;
 __host__ __device__ constexpr size_t delta_block_floats(int DP, int nsl) { return (size_t)49 * DP + (size_t)nsl * 512; }
 
 template <typename T, int KT>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, 2)
 delta_channel_block_kernel(const qspec_delta_channel_args a, const int* __restrict__ block_rows, float* __restrict__ blocks, int DP) {
-  pdl_enter();
+  pdl_enter_hold();
   extern __shared__ __align__(16) float sm_db[];
   const int x = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int i0 = block_rows[x];
@@ -412,10 +412,16 @@ delta_channel_block_kernel(const qspec_delta_channel_args a, const int* __restri
       float w[KT ? KT : 1], in[DBLK + (KT ? KT : 1) - 1];
 #pragma unroll
       for (int j = 0; j < KT; ++j) { const int jr = j - (KT - 1 - K1); w[j] = jr >= 0 ? a.conv_w[(size_t)jr * C + ch] : 0.f; }
+      // the block's rows: every load is issued before the first is used (rows past the end repeat the last one and are dropped)
+      const T* src = (const T*)a.p + (size_t)i0 * a.ld + ch;
 #pragma unroll
-      for (int t = 0; t < DBLK + KT - 1; ++t) {
-        const int back = KT - 1 - t;                              // positions before the block's first token
-        in[t] = (back > K1 || -back >= nb) ? 0.f : cv.get(mt.pos - back, ch);
+      for (int t = 0; t < DBLK; ++t) in[t + KT - 1] = to_f(src[(size_t)min(t, nb - 1) * a.ld]);
+      if (i0 == mt.seg_begin) {                                   // the rows before the step
+#pragma unroll
+        for (int t = 0; t < KT - 1; ++t) in[t] = t < KT - 1 - K1 ? 0.f : cv.get(mt.pos - (KT - 1 - t), ch);
+      } else {
+#pragma unroll
+        for (int t = 0; t < KT - 1; ++t) in[t] = to_f(*(src - (size_t)(KT - 1 - t) * a.ld));
       }
 #pragma unroll
       for (int t = 0; t < DBLK; ++t) {
@@ -440,7 +446,7 @@ delta_channel_block_kernel(const qspec_delta_channel_args a, const int* __restri
     const float db = ok ? a.dt_bias[h * D + c] : 0.f;
     float z[DBLK];
 #pragma unroll
-    for (int t = 0; t < DBLK; ++t) z[t] = ok && t < nb ? a.decay[(size_t)(i0 + t) * a.decay_ld + (size_t)h * D + c] : 0.f;
+    for (int t = 0; t < DBLK; ++t) z[t] = a.decay[(size_t)(i0 + min(t, nb - 1)) * a.decay_ld + (size_t)h * D + (ok ? c : 0)];
 #pragma unroll
     for (int t = 0; t < DBLK; ++t) sG[t * DS + c] = ok && t < nb ? expf(-rate * softplus_f(z[t] + db)) : 1.f;
   }
@@ -460,33 +466,47 @@ delta_channel_block_kernel(const qspec_delta_channel_args a, const int* __restri
   __syncthreads();
   // ---- A and B: 16 lanes per s; the running product k_s g_(s+1) .. g_t meets k_t and q_t
   {
-    const int s = tid >> 4, l = tid & 15, s0 = 2 * warp;
+    const int s = tid >> 4, l = tid & 15;
     float4 w[4];
 #pragma unroll
     for (int m = 0; m < 4; ++m)
       w[m] = m * 64 < DP ? *reinterpret_cast<const float4*>(sK + s * DS + m * 64 + 4 * l) : make_float4(0.f, 0.f, 0.f, 0.f);
-    for (int t = s0; t < nb; ++t) {
-      float dk = 0.f, dq = 0.f;
+    for (int t0 = (2 * warp) & ~3; t0 < nb; t0 += 4) {            // four tokens' sums at a time
+      float p[8];                                                 // [token][key, query]
 #pragma unroll
-      for (int m = 0; m < 4; ++m) {
-        if (m * 64 >= DP) break;
-        const int at = t * DS + m * 64 + 4 * l;
-        const float4 k = *reinterpret_cast<const float4*>(sK + at), q = *reinterpret_cast<const float4*>(sQ + at);
-        if (t > s) {
-          const float4 g = *reinterpret_cast<const float4*>(sG + at);
-          w[m].x *= g.x; w[m].y *= g.y; w[m].z *= g.z; w[m].w *= g.w;
+      for (int u = 0; u < 4; ++u) {
+        const int t = t0 + u;
+        float dk = 0.f, dq = 0.f;
+#pragma unroll
+        for (int m = 0; m < 4; ++m) {
+          if (m * 64 >= DP) break;
+          const int at = t * DS + m * 64 + 4 * l;
+          const float4 k = *reinterpret_cast<const float4*>(sK + at), q = *reinterpret_cast<const float4*>(sQ + at);
+          if (t > s) {
+            const float4 g = *reinterpret_cast<const float4*>(sG + at);
+            w[m].x *= g.x; w[m].y *= g.y; w[m].z *= g.z; w[m].w *= g.w;
+          }
+          dk += (w[m].x * k.x + w[m].y * k.y) + (w[m].z * k.z + w[m].w * k.w);
+          dq += (w[m].x * q.x + w[m].y * q.y) + (w[m].z * q.z + w[m].w * q.w);
         }
-        dk += (w[m].x * k.x + w[m].y * k.y) + (w[m].z * k.z + w[m].w * k.w);
-        dq += (w[m].x * q.x + w[m].y * q.y) + (w[m].z * q.z + w[m].w * q.w);
+        p[2 * u] = dk;
+        p[2 * u + 1] = dq;
       }
+      // eight sums over 16 lanes by halving exchanges: lane bits 3, 2, 1 select the sum a lane ends with, bit 0 adds the last two
 #pragma unroll
-      for (int off = 1; off < 16; off <<= 1) {
-        dk += __shfl_xor_sync(0xffffffffu, dk, off);
-        dq += __shfl_xor_sync(0xffffffffu, dq, off);
+      for (int n = 4; n >= 1; n >>= 1) {
+        const bool hi = (l & (2 * n)) != 0;
+#pragma unroll
+        for (int j = 0; j < n; ++j) {
+          const float send = hi ? p[j] : p[j + n], keep = hi ? p[j + n] : p[j];
+          p[j] = keep + __shfl_xor_sync(0xffffffffu, send, 2 * n);
+        }
       }
-      if (l == 0 && t >= s) {
-        if (t > s) sA[s * 16 + t] = sbeta[t] * dk;
-        sB[t * 16 + s] = dq;
+      p[0] += __shfl_xor_sync(0xffffffffu, p[0], 1);
+      const int t = t0 + (l >> 2);                                // sum index l >> 1 = 2 u + (0 key, 1 query)
+      if ((l & 1) == 0 && t >= s && t < nb) {
+        if (l & 2) sB[t * 16 + s] = p[0];
+        else if (t > s) sA[s * 16 + t] = sbeta[t] * p[0];
       }
     }
   }
