@@ -60,6 +60,11 @@ template <int VEC> __global__ void __launch_bounds__(256) softcap_kernel(float* 
   }
 }
 
+// silu of a convolution's result: in bfloat16 mode (the inputs are bfloat16 roundings, relative 4e-3) the exponential and the
+// division run on the special-function unit
+template <typename T> __device__ __forceinline__ float silu_act(float z) { return silu_f(z); }
+template <> __device__ __forceinline__ float silu_act<bf16_t>(float z) { return __fdividef(z, 1.0f + __expf(-z)); }
+
 // ---- inputs of a short causal convolution -------------------------------------------------------------------------------------
 // The input of channel c at position sp: a row of the step, a row of the slot's tail (the last K1 inputs before the step), or zero
 // before the sequence's start.
@@ -270,7 +275,7 @@ delta_channel_token_kernel(const qspec_delta_channel_args a, int max_len) {
       float acc = 0.f;
       for (int j = 0; j <= K1; ++j) acc += a.conv_w[(size_t)j * C + ch] * cv.get(pos - K1 + j, ch);
       if (tt == len - 1) cv.write_tail(tnew, pos, ch);            // every head of a group writes the same query / key tail
-      return silu_f(acc);
+      return silu_act<T>(acc);
     };
     if (warp < 2) {                                               // unit query (warp 0) and key (warp 1)
       float* dst = warp ? sk : sq;
@@ -428,14 +433,14 @@ delta_channel_block_kernel(const qspec_delta_channel_args a, const int* __restri
         float acc = 0.f;
 #pragma unroll
         for (int j = 0; j < KT; ++j) acc += w[j] * in[t + j];
-        dst[t * ds] = t < nb ? silu_f(acc) : 0.f;
+        dst[t * ds] = t < nb ? silu_act<T>(acc) : 0.f;
       }
     } else {
       for (int t = 0; t < DBLK; ++t) {
         float acc = 0.f;
         if (t < nb)
           for (int j = 0; j <= K1; ++j) acc += a.conv_w[(size_t)j * C + ch] * cv.get(mt.pos + t - K1 + j, ch);
-        dst[t * ds] = silu_f(acc);
+        dst[t * ds] = silu_act<T>(acc);
       }
     }
     if (last && (kind == 2 || h % rep == 0)) cv.write_tail(tnew, mt.pos + nb - 1, ch);
@@ -606,13 +611,14 @@ delta_channel_block_kernel(const qspec_delta_channel_args a, const int* __restri
 
 __device__ __forceinline__ unsigned long long f2_dup(float v) { return pack_f2(v, v); }
 
-// The part in sequence order. One CTA of four warps per (segment, head, 16 value columns); a warp owns four columns, its lanes own
-// key channels hx * 64 + 2 lane + {0, 1}. Products run as packed pairs of float32 (two tokens of the block at a time, the state kept
-// as duplicated pairs). The sums over the channels of 16 (kind, token pair) x 4 columns x 2 tokens are taken by halving exchanges:
-// accumulator slot j of lane L belongs to row j ^ (L >> 1), so that every exchange sends the slots the lane does not keep and no
-// selection is needed. The blocks' operands arrive one block ahead by cp.async.
+// The part in sequence order. One CTA of eight warps per (segment, head, 16 value columns); two warps share four columns, one for the
+// corrections (Wk) and one for the read-outs (Qk), each with its own copy of the columns; lanes own key channels hx * 64 + 2 lane +
+// {0, 1}. Products run as packed pairs of float32 (two tokens of the block at a time, the state kept
+// as duplicated pairs). The sums over the channels of 8 token pairs x 4 columns x 2 tokens are taken by halving exchanges: accumulator slot j of
+// lane L belongs to token pair j ^ (L >> 2), so that the exchanges over token pairs send the slots the lane does not keep and need no
+// selection. The blocks' operands arrive one block ahead by cp.async.
 template <int NHR>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(256)
 delta_channel_scan_kernel(const qspec_delta_channel_args a, const int* __restrict__ long_starts, const int* __restrict__ long_block0,
                           const float* __restrict__ blocks, float* __restrict__ o) {
   pdl_enter();
@@ -623,14 +629,14 @@ delta_channel_scan_kernel(const qspec_delta_channel_args a, const int* __restric
   const int i0 = long_starts[blockIdx.x], x0 = long_block0[blockIdx.x], h = blockIdx.y, sl = blockIdx.z;
   const TokMeta mt = load_meta(a.meta, a.ntok, i0);
   const int H = a.H, D = a.D, DV = a.DV, nsl = gridDim.z;
-  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, xl = lane >> 1;
+  const int tid = threadIdx.x, lane = tid & 31, warp = (tid >> 5) & 3, kind = tid >> 7, xl = lane >> 2;
   const int len = mt.seg_end - mt.seg_begin, nblk = (len + DBLK - 1) / DBLK, c0 = sl * 16 + warp * 4;
   const size_t bf = delta_block_floats(DP, nsl);
   auto stage = [&](int buf, int b) {
     const float* src = blocks + ((size_t)(x0 + b) * H + h) * bf;
     float* dst = sm_ds + buf * NF;
-    for (int e = tid; e < 49 * DP / 4; e += 128) cp_async_16z(dst + 4 * e, src + 4 * e, true);
-    cp_async_16z(dst + 49 * DP + 4 * tid, src + 49 * DP + (size_t)sl * 512 + 4 * tid, true);       // 512 floats = 128 x 16 bytes
+    for (int e = tid; e < 49 * DP / 4; e += 256) cp_async_16z(dst + 4 * e, src + 4 * e, true);
+    if (tid < 128) cp_async_16z(dst + 49 * DP + 4 * tid, src + 49 * DP + (size_t)sl * 512 + 4 * tid, true);       // 512 floats = 128 x 16 bytes
     cp_async_commit();
   };
   stage(0, 0);
@@ -646,72 +652,68 @@ delta_channel_scan_kernel(const qspec_delta_channel_args a, const int* __restric
     }
   for (int b = 0; b < nblk; ++b) {
     const int buf = b & 1;
-    if (b + 1 < nblk) { stage(buf ^ 1, b + 1); cp_async_wait<1>(); } else cp_async_wait<0>();
-    __syncthreads();
+    cp_async_wait<0>();
+    __syncthreads();                                              // block b has arrived, and nobody reads block b - 1 any more
+    if (b + 1 < nblk) stage(buf ^ 1, b + 1);
     const float* B = sm_ds + buf * NF;
-    unsigned long long acc[16][4];
+    unsigned long long acc[8][4];
 #pragma unroll
-    for (int j = 0; j < 16; ++j)
+    for (int j = 0; j < 8; ++j)
 #pragma unroll
       for (int c = 0; c < 4; ++c) acc[j][c] = 0ull;
     const uint32_t perm = (uint32_t)(xl * ROW * 4 + lane * 16);   // a row is a power of two of bytes: row j ^ xl = (j rows) ^ (xl rows)
-    const char* Bc = reinterpret_cast<const char*>(B);
+    const char* Bc = reinterpret_cast<const char*>(B + kind * 8 * ROW);
 #pragma unroll
     for (int hx = 0; hx < NHR; ++hx)
 #pragma unroll
-      for (int j = 0; j < 16; ++j) {
+      for (int j = 0; j < 8; ++j) {
         const ulonglong2 w = *reinterpret_cast<const ulonglong2*>(Bc + (((uint32_t)(j * ROW * 4) ^ perm) + hx * 512));
 #pragma unroll
-        for (int c = 0; c < 4; ++c) {
-          acc[j][c] = ffma2_rn(w.x, S[hx][0][c], acc[j][c]);
-          acc[j][c] = ffma2_rn(w.y, S[hx][1][c], acc[j][c]);
-        }
-      }
-    float v[16][4][2];
+        for (int c = 0; c < 4; ++c) acc[j][c] = ffma2_rn(w.x, S[hx][0][c], acc[j][c]);
 #pragma unroll
-    for (int j = 0; j < 16; ++j)
+        for (int c = 0; c < 4; ++c) acc[j][c] = ffma2_rn(w.y, S[hx][1][c], acc[j][c]);
+      }
+    float v[8][4][2];
+#pragma unroll
+    for (int j = 0; j < 8; ++j)
 #pragma unroll
       for (int c = 0; c < 4; ++c) { const float2 f = unpack_f2(acc[j][c]); v[j][c][0] = f.x; v[j][c][1] = f.y; }
 #pragma unroll
-    for (int n = 8; n >= 1; n >>= 1)                              // lane bit of the exchange: n << 1
+    for (int n = 4; n >= 1; n >>= 1)                              // lane bit of the exchange: n << 2
 #pragma unroll
       for (int j = 0; j < n; ++j)
 #pragma unroll
         for (int c = 0; c < 4; ++c) {
-          v[j][c][0] += __shfl_xor_sync(0xffffffffu, v[j + n][c][0], n << 1);
-          v[j][c][1] += __shfl_xor_sync(0xffffffffu, v[j + n][c][1], n << 1);
+          v[j][c][0] += __shfl_xor_sync(0xffffffffu, v[j + n][c][0], n << 2);
+          v[j][c][1] += __shfl_xor_sync(0xffffffffu, v[j + n][c][1], n << 2);
         }
-    const int hb = lane & 1;                                      // this lane keeps columns 2 hb, 2 hb + 1
-    float r[2][2];
+    // two more exchanges: over the column pairs (lane bit 1), then over the columns of a pair (lane bit 0)
+    const int hp = (lane >> 1) & 1, hc = lane & 1;
+    float r[2], m[2][2];
 #pragma unroll
     for (int c = 0; c < 2; ++c)
 #pragma unroll
       for (int par = 0; par < 2; ++par) {
-        const float send = hb ? v[0][c][par] : v[0][2 + c][par], keep = hb ? v[0][2 + c][par] : v[0][c][par];
-        r[c][par] = keep + __shfl_xor_sync(0xffffffffu, send, 1);
+        const float send = hp ? v[0][c][par] : v[0][2 + c][par], keep = hp ? v[0][2 + c][par] : v[0][c][par];
+        m[c][par] = keep + __shfl_xor_sync(0xffffffffu, send, 2);
       }
-    // lanes 0 .. 15 hold S0^T Wk of token pair xl, lanes 16 .. 31 S0^T Qk of token pair xl - 8
+#pragma unroll
+    for (int par = 0; par < 2; ++par) {
+      const float send = hc ? m[0][par] : m[1][par], keep = hc ? m[1][par] : m[0][par];
+      r[par] = keep + __shfl_xor_sync(0xffffffffu, send, 1);
+    }
+    // this lane holds the two tokens of pair xl for column 2 hp + hc of its warp
     {
-      const int tp = xl & 7, kind = xl >> 3, cl = warp * 4 + 2 * hb;
+      const int cl = warp * 4 + (lane & 3);
       const float* uo = B + 49 * DP + kind * 256 + cl;
 #pragma unroll
       for (int par = 0; par < 2; ++par) {
-        const int t = 2 * tp + par;
-        const float2 base = *reinterpret_cast<const float2*>(uo + t * 16);
-        if (kind == 0) {
-          su[warp][tp][2 * hb][par] = base.x - r[0][par];
-          su[warp][tp][2 * hb + 1][par] = base.y - r[1][par];
-        } else {
-          const int row = i0 + b * DBLK + t, col = sl * 16 + cl;
-          if (b * DBLK + t < len) {
-            float* dst = o + ((size_t)row * H + h) * DV + col;
-            if (col < DV) dst[0] = base.x + r[0][par];
-            if (col + 1 < DV) dst[1] = base.y + r[1][par];
-          }
-        }
+        const int t = 2 * xl + par;
+        if (kind == 0) su[warp][xl][lane & 3][par] = uo[t * 16] - r[par];
+        else if (b * DBLK + t < len && sl * 16 + cl < DV) o[((size_t)(i0 + b * DBLK + t) * H + h) * DV + sl * 16 + cl] = uo[t * 16] + r[par];
       }
     }
-    __syncwarp();
+    __syncthreads();                                              // the corrections are complete
     unsigned long long add[NHR][2][4];
 #pragma unroll
     for (int hx = 0; hx < NHR; ++hx)
@@ -746,8 +748,8 @@ delta_channel_scan_kernel(const qspec_delta_channel_args a, const int* __restric
           S[hx][e][c] = f2_dup((e ? g.y : g.x) * unpack_f2(S[hx][e][c]).x + (ad.x + ad.y));
         }
     }
-    __syncthreads();                                              // the buffer is refilled two blocks later
   }
+  if (kind) return;                                               // both copies are the same
 #pragma unroll
   for (int hx = 0; hx < NHR; ++hx)
 #pragma unroll
@@ -931,7 +933,7 @@ static int launch_delta_scan_blocks(const qspec_delta_channel_args& a, const int
     QSPEC_CUDA(cudaFuncSetAttribute(delta_channel_scan_kernel<NHR>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     configured = true;
   }
-  launch_pdl(delta_channel_scan_kernel<NHR>, dim3(nlong, a.H, (a.DV + 15) / 16), dim3(128), smem, st, a, long_starts, long_block0, blocks, o);
+  launch_pdl(delta_channel_scan_kernel<NHR>, dim3(nlong, a.H, (a.DV + 15) / 16), dim3(256), smem, st, a, long_starts, long_block0, blocks, o);
   QSPEC_CHECK_LAUNCH(1);
   return QSPEC_OK;
 }
