@@ -178,7 +178,7 @@ typedef struct qspec_window_attn_args {
                           j < keep_first) and their ring rows are never reused: row = j for j < cap, otherwise keep_first +
                           (j - keep_first) % (cap - keep_first). cap >= keep_first + window - 1 + (tokens of one sequence in a step). */
   long long out_tok_stride;   /* elements from one token's output row to the next; 0: H * DV */
-  float out_scale;     /* factor on the output; 0: one */
+  float out_scale;     /* factor on the output */
 } qspec_window_attn_args;
 int qspec_seq_window_attention(const qspec_window_attn_args* args, int dtype, void* stream);
 

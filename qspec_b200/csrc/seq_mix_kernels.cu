@@ -723,7 +723,7 @@ static int launch_window_attn(const qspec_window_attn_args* a, cudaStream_t st) 
              a->qb, a->qb_tok_stride, a->qb_head_stride, a->DB, (const T*)a->k, a->k_slot_stride, a->k_row_stride, a->k_head_stride,
              (const T*)a->v, a->v_slot_stride, a->v_row_stride, a->v_head_stride, a->DV, a->sink, (const T*)a->gate, a->gate_ld, a->gate_per_head, (T*)a->out,
              a->meta, a->ntok, a->H, a->G, a->window, a->cap, a->scale, a->keep_first,
-             a->out_tok_stride ? a->out_tok_stride : (long long)a->H * a->DV, a->out_scale != 0.f ? a->out_scale : 1.0f);
+             a->out_tok_stride ? a->out_tok_stride : (long long)a->H * a->DV, a->out_scale);
   QSPEC_CHECK_LAUNCH(1);
   return QSPEC_OK;
 }

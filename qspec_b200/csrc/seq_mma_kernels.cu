@@ -1684,7 +1684,7 @@ int prompt_attention_mma(const qspec_window_attn_args* p, const void* kB, long l
   a.out = (bf16*)p->out; a.out_hs = DV; a.meta = p->meta; a.ntok = p->ntok; a.H = p->H; a.G = p->G; a.window = p->window; a.cap = p->cap;
   a.scale = p->scale; a.token_rows = 1;
   a.keep = p->keep_first; a.out_ts = p->out_tok_stride ? p->out_tok_stride : (long long)p->H * DV;
-  a.out_scale = p->out_scale != 0.f ? p->out_scale : 1.0f;
+  a.out_scale = p->out_scale;
   if (DB) return launch_prompt_attn<128, 64, 128>(a, slot, pos0, st);
   if (DA == 128) return launch_prompt_attn<128, 0, 128>(a, slot, pos0, st);
   return launch_prompt_attn<64, 0, 64>(a, slot, pos0, st);
@@ -1733,7 +1733,7 @@ int window_attention_mma(const qspec_window_attn_args* p, const void* kB, long l
   a.out = (bf16*)p->out; a.out_hs = DV; a.meta = p->meta; a.ntok = p->ntok; a.H = p->H; a.G = p->G; a.window = p->window; a.cap = p->cap;
   a.scale = p->scale; a.token_rows = token_rows;
   a.keep = p->keep_first; a.out_ts = p->out_tok_stride ? p->out_tok_stride : (long long)p->H * DV;
-  a.out_scale = p->out_scale != 0.f ? p->out_scale : 1.0f;
+  a.out_scale = p->out_scale;
   // a latent cache read in the absorbed form (keys and values are the same rows): the CTA-level kernel; QSPEC_SEQ_LATENT=sliced
   // keeps the form with one CTA per slice of 128 value columns, for comparison
   static const bool sliced = [] { const char* v = getenv("QSPEC_SEQ_LATENT"); return v && !strcmp(v, "sliced"); }();

@@ -379,3 +379,314 @@ def test_a_key_that_stands_out_at_every_edge(form, dtype, sizes, place):
         _attend(form, dev(q[n - count:]), ck, cv, out, meta, w, 1.0, keep_first=kf)
         close(out, want[n - count:], dtype, scale=float(want[n - count:].abs().max()))
         assert (float(out[-1, 1].float().mean()) > 2.0) == seen
+
+
+# ---------------------------------------------------------------------------------------------------------------------
+# whole models through the scheduler
+# ---------------------------------------------------------------------------------------------------------------------
+def attention(heads=4, kv_heads=2, dim=16, scale=0.3, window=20, keep=3, dims=None, base=500.0, scaling=None):
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": scale, "mask": {"size": window, "keep_first": keep},
+         "rot": {"base": base, "dims": dim if dims is None else dims}}
+    if scaling:
+        m["rot"]["scaling"] = scaling
+    return {"type": "attention", "mixer": m}
+
+
+def parallel(left=(4, 2, 16, 12), lconv=3, temp=(0.3, 8), right=(4, 2, 12, 10), rconv=4, scales=(0.8, 1.25), scale=0.25):
+    lh, lg, ld, lv = left
+    rh, rg, rd, rv = right
+    lm = {"heads": lh, "kv_heads": lg, "dim": ld, "vdim": lv, "conv": lconv, "scale": scale}
+    if temp:
+        lm["q_temp"] = {"coef": temp[0], "every": temp[1]}
+    return {"type": "parallel", "mixer": {"left": lm, "right": {"heads": rh, "kv_heads": rg, "dim": rd, "vdim": rv, "conv": rconv},
+                                          "left_scale": scales[0], "right_scale": scales[1]}}
+
+
+def moe(ff=24, experts=8, top=3, count=4, keep=2):
+    return {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top, "groups": {"count": count, "keep": keep}}}
+
+
+def config(layers, width=64, vocab=97, eps=1e-5, softcap=12.0):
+    return {"architecture": "Legavik", "vocab": vocab, "width": width, "norm": {"eps": eps}, "logit_softcap": softcap, "layers": layers}
+
+
+STRETCH = {"factor": 4.0, "original": 64, "fast": 8.0, "slow": 1.0}
+CONFIGS = {
+    # both mixers, grouped heads on every side, windows shorter and longer than the portions
+    "mixed": (config([dict(attention(scaling=STRETCH), mlp=moe()), dict(parallel(), mlp=moe(ff=16, experts=6, top=2, count=2, keep=1)),
+                      dict(attention(heads=6, kv_heads=1, dim=8, dims=4, window=33, keep=0), mlp=None),
+                      dict(parallel(left=(2, 2, 24, 8), right=(6, 3, 8, 6), lconv=2, rconv=2), mlp=moe())]), 5, 7),
+    # nothing divisible by anything: one head, all heads on one key, one-tap and long convolutions, no temperature, no rotation, one
+    # expert per token, as many chosen as there are, a window of one token, layers that open with a parallel mixer
+    "odd": (config([dict(parallel(left=(3, 3, 10, 7), right=(1, 1, 33, 7), lconv=1, rconv=5, temp=None, scales=(1.0, 1.0)), mlp=None),
+                    dict(attention(heads=3, kv_heads=1, dim=10, dims=0, window=1, keep=2), mlp=moe(ff=13, experts=5, top=1, count=1, keep=1)),
+                    dict(parallel(left=(1, 1, 6, 9), right=(3, 1, 5, 17), lconv=6, rconv=1, temp=(0.5, 1)), mlp=moe(ff=9, experts=3, top=3, count=3, keep=3)),
+                    dict(attention(heads=5, kv_heads=5, dim=7, dims=2, base=37.0, window=9, keep=11), mlp=None)],
+                   width=50, vocab=33, eps=1e-6, softcap=5.0), 3, 1),
+    # head sizes of the tensor-core forms, a key size above 128 in the recurrence, values wider than one pass
+    "wide": (config([dict(attention(heads=4, kv_heads=2, dim=64, dims=32, scaling=STRETCH, scale=0.12, window=48, keep=4), mlp=moe(ff=32)),
+                     dict(parallel(left=(4, 1, 64, 128), right=(2, 1, 130, 40), scale=0.1), mlp=None),
+                     dict(parallel(left=(2, 2, 128, 64), right=(2, 2, 24, 136), scale=0.08), mlp=moe(ff=32))], width=96, softcap=20.0), 16, 8),
+}
+
+
+def build(name, dtype, seed=0, n_slots=3, max_step_tokens=64, max_seq_tokens=256):
+    _cuda()
+    from qspec_b200.legavik import LegavikConfig, LegavikModel, random_weights
+    from qspec_b200.scheduler import Scheduler
+    d, rd, rg = CONFIGS[name]
+    cfg = LegavikConfig.from_dict(d)
+    w = random_weights(cfg.with_ranks(decay_rank=rd, gate_rank=rg), seed)
+    model = LegavikModel(cfg, w, dtype=dtype, device="cuda", n_slots=n_slots, max_step_tokens=max_step_tokens, max_seq_tokens=max_seq_tokens)
+    model.prompt_tiles_min_ctas = 2                        # short test prompts take the tile form too
+    return d, w, model, Scheduler(model)
+
+
+def tokens(n, vocab, seed):
+    return torch.randint(0, vocab, (n,), generator=torch.Generator().manual_seed(seed)).tolist()
+
+
+def close_logits(got, ref, dtype, same_format=False):
+    """Per position: root mean square over the vocabulary of the difference (mean taken off), relative to the spread of the
+    logits. float32 against the plain implementation: rounding level. bfloat16 against the plain implementation: what an 8-bit
+    mantissa leaves, with a few positions further off where two experts' scores are nearly equal. same_format: bfloat16 against
+    bfloat16 logits of the same model fed another way."""
+    ref = ref.to(F64)
+    d = got.detach().cpu().to(F64) - ref
+    d = d - d.mean(-1, keepdim=True)
+    spread = float((ref - ref.mean(-1, keepdim=True)).pow(2).mean().sqrt())
+    rows = d.pow(2).mean(-1).sqrt() / spread
+    if dtype == F32:
+        assert float(rows.median()) <= 1e-5, f"median position: {float(rows.median()):.3g} of the logits' spread"
+        assert float(rows.max()) <= 3e-4, f"worst position: {float(rows.max()):.3g} of the logits' spread"
+        return
+    bound = 1.5e-2 if same_format else 3e-2
+    assert float(rows.median()) <= bound, f"median position: {float(rows.median()):.3g} of the logits' spread"
+    over = float((rows > 0.1).float().mean())
+    assert over <= 0.1, f"{over:.1%} of the positions are off by more than 10% of the logits' spread"
+
+
+_PLAIN = {}
+
+
+def plain(name, toks, seed=0, layers=None):
+    """The plain implementation's logits, computed once per model and sequence."""
+    key = (name, seed, tuple(toks))
+    if key not in _PLAIN:
+        from qspec_b200.legavik import LegavikConfig, random_weights
+        d, rd, rg = CONFIGS[name]
+        lay = []
+        _PLAIN[key] = (O.forward(d, random_weights(LegavikConfig.from_dict(d).with_ranks(decay_rank=rd, gate_rank=rg), seed), toks, lay), lay)
+    if layers is not None:
+        layers.extend(_PLAIN[key][1])
+    return _PLAIN[key][0]
+
+
+def reference_logits(name, toks, dtype):
+    """float32: the plain implementation. bfloat16: the same weights in a second model that takes the prompt whole, after that
+    has been held against the plain implementation."""
+    ref = plain(name, toks)
+    if dtype == F32:
+        return ref
+    _, _, _, s = build(name, dtype, max_step_tokens=256)
+    whole = s.feed([("whole", toks, list(range(len(toks))))]).float().cpu()
+    close_logits(whole, ref, dtype)
+    return whole
+
+
+@pytest.mark.parametrize("dtype", [F32, BF16])
+@pytest.mark.parametrize("name", list(CONFIGS))
+def test_whole_prompt_matches_the_plain_implementation(name, dtype):
+    cfg, w, model, s = build(name, dtype, max_step_tokens=128)
+    toks = tokens(90, cfg["vocab"], 1)
+    lay = []
+    ref = plain(name, toks, layers=lay)
+    close_logits(s.feed([("a", toks, list(range(len(toks))))]), ref, dtype)
+    if dtype == F32:                                       # residual stream after every layer
+        meta = s.table.plan([("b", len(toks))])
+        tr = []
+        model.forward_batch(torch.tensor(toks, dtype=torch.int32, device="cuda"), meta, trace=tr)
+        assert len(tr) == len(lay) == len(cfg["layers"])
+        for a, b in zip(tr, lay):
+            close(a, b, F32)
+
+
+@pytest.mark.parametrize("dtype", [F32, BF16])
+@pytest.mark.parametrize("name", list(CONFIGS))
+def test_decoding_and_portions_equal_the_whole_prompt(name, dtype):
+    """Token by token from the first token on; a prompt then 40 single tokens; portions of 2, 3, 1, 7, ... tokens; a step
+    longer than the model's step size (cut inside the step function)."""
+    cfg, w, model, s = build(name, dtype, max_step_tokens=16)
+    toks = tokens(90, cfg["vocab"], 1)
+    ref = reference_logits(name, toks, dtype)
+    schedules = {"single": [1] * len(toks), "prompt+decode": [16, 16, 16, 2] + [1] * 40, "twos": [2] * 45,
+                 "portions": [2, 3, 1, 7, 2, 2, 13, 5, 2, 16, 9, 11, 14, 3], "one step": [len(toks)]}
+    for label, cuts in schedules.items():
+        assert sum(cuts) == len(toks)
+        at, rows = 0, []
+        for n in cuts:
+            rows.append(s.feed([(label, toks[at:at + n], list(range(n)))]))
+            at += n
+        s.release(label)
+        close_logits(torch.cat(rows), ref, dtype, same_format=True)
+
+
+@pytest.mark.parametrize("name", ["mixed", "wide"])
+@pytest.mark.parametrize("dtype", [F32, BF16])
+def test_mixed_batches_equal_each_request_alone_and_slots_are_reused(name, dtype):
+    """Three requests of unequal length advance together -- a prompt portion next to single tokens next to a request that
+    starts late in a slot another request has just given back -- and each must see what it sees alone."""
+    cfg, w, model, s = build(name, dtype, n_slots=2, max_step_tokens=48)
+    seqs = {"a": tokens(60, cfg["vocab"], 11), "b": tokens(23, cfg["vocab"], 12), "c": tokens(41, cfg["vocab"], 13)}
+    alone = {}
+    for rid, toks in seqs.items():
+        alone[rid] = s.feed([(rid, toks, list(range(len(toks))))]).float().cpu()
+        s.release(rid)
+        if dtype == F32:
+            close_logits(alone[rid], plain(name, toks), dtype)
+    sched = [{"a": 7, "b": 20}, {"a": 1, "b": 1}, {"a": 30, "b": 2}, {"a": 1}, {"a": 1, "c": 9}, {"a": 2, "c": 1}, {"a": 18, "c": 30}, {"c": 1}]
+    at = {k: 0 for k in seqs}
+    got = {k: [] for k in seqs}
+    for stepn, st in enumerate(sched):
+        entries = [(rid, seqs[rid][at[rid]:at[rid] + n], list(range(n))) for rid, n in st.items()]
+        out = s.feed(entries)
+        o = 0
+        for rid, n in st.items():
+            got[rid].append(out[o:o + n].float().cpu())
+            o += n
+            at[rid] += n
+        if stepn == 2:
+            assert at["b"] == len(seqs["b"])
+            s.release("b")                                  # request c takes this slot in the step after next
+    for rid in seqs:
+        assert at[rid] == len(seqs[rid])
+        close_logits(torch.cat(got[rid]), alone[rid], dtype, same_format=True)
+
+
+def test_batch_composition_changes_nothing_in_float32():
+    """The same token of the same request, once alone in its step and once between two other requests: every kernel assigns work
+    by position and size alone, so the logits agree to the last rounding of the vendor's matrix products."""
+    cfg, w, model, s = build("odd", F32, n_slots=3, max_step_tokens=64)
+    a, b, c = tokens(20, cfg["vocab"], 21), tokens(9, cfg["vocab"], 22), tokens(14, cfg["vocab"], 23)
+    assert s.feed([("a", a[:19], []), ("b", b[:8], []), ("c", c[:13], [])]).shape[0] == 0
+    mixed = s.feed([("b", b[8:], [0]), ("a", a[19:], [0]), ("c", c[13:], [0])])[1].float().cpu()
+    for rid in "abc":
+        s.release(rid)
+    s.feed([("a", a[:19], [])])
+    alone = s.feed([("a", a[19:], [0])])[0].float().cpu()
+    assert float((mixed - alone).abs().max()) <= 2e-5 * float(alone.abs().max())
+
+
+@pytest.mark.parametrize("half", ["left", "right"])
+def test_each_half_of_a_parallel_layer_alone(half):
+    """With one half's scale at zero the other one is all there is: the silent half's weights must not matter, its state and
+    bias included."""
+    from qspec_b200.legavik import LegavikConfig, LegavikModel, random_weights
+    from qspec_b200.scheduler import Scheduler
+    _cuda()
+    scales = (1.5, 0.0) if half == "left" else (0.0, 1.5)
+    d = config([dict(parallel(scales=scales), mlp=None), dict(parallel(scales=scales), mlp=moe())])
+    w = random_weights(LegavikConfig.from_dict(d).with_ranks(decay_rank=5, gate_rank=7), 4)
+    toks = tokens(40, 97, 4)
+    ref = O.forward(d, w, toks)
+    other = "right" if half == "left" else "left"
+    w2 = {k: (v.flip(0) * 2.0 if f".{other}." in k and v.dim() else v) for k, v in w.items()}
+    for ww in (w, w2):
+        m = LegavikModel(LegavikConfig.from_dict(d), ww, dtype=F32, device="cuda", n_slots=1, max_step_tokens=20, max_seq_tokens=64)
+        close_logits(Scheduler(m).feed([("a", toks, list(range(40)))]), ref, F32)
+
+
+def test_the_ring_of_a_window_layer_is_short_and_keeps_its_first_rows():
+    """A model of window layers alone does not bound the sequence: its rings hold the kept rows, the window and a step; far beyond
+    them, prompts and decoding still equal the plain implementation."""
+    from qspec_b200.legavik import LegavikConfig, LegavikModel, random_weights
+    from qspec_b200.scheduler import Scheduler
+    _cuda()
+    d = config([dict(attention(window=12, keep=3, scaling=STRETCH), mlp=None), dict(attention(window=5, keep=6, heads=2, kv_heads=2), mlp=moe())])
+    w = random_weights(LegavikConfig.from_dict(d), 6)
+    m = LegavikModel(LegavikConfig.from_dict(d), w, dtype=F32, device="cuda", n_slots=2, max_step_tokens=10)
+    assert m.max_seq_len is None and m.cache_k[0].shape[1] == 3 + 12 - 1 + 10 and m.cache_k[1].shape[1] == 6 + 5 - 1 + 10
+    s = Scheduler(m)
+    toks = tokens(160, 97, 7)
+    ref = O.forward(d, w, toks)
+    for label, cuts in (("whole", [160]), ("decode", [70] + [1] * 90), ("portions", [10, 2, 3, 10, 7] * 5)):
+        at, rows = 0, []
+        for n in cuts:
+            rows.append(s.feed([(label, toks[at:at + n], list(range(n)))]))
+            at += n
+        close_logits(torch.cat(rows), ref, F32)
+        s.release(label)
+
+
+def test_the_cache_bounds_the_sequence_and_the_scheduler_refuses_more():
+    cfg, w, model, s = build("mixed", BF16, max_seq_tokens=40)
+    s.feed([("a", tokens(40, cfg["vocab"], 5), [39])])
+    with pytest.raises(RuntimeError):
+        s.feed([("a", [1], [0])])
+
+
+def test_long_decoding():
+    """A short prompt, then 230 single tokens: windows pass over decoded tokens several times, the recurrences' states and the growing
+    cache, against the plain implementation."""
+    cfg, w, model, s = build("mixed", F32, max_step_tokens=8, max_seq_tokens=512)
+    toks = tokens(250, cfg["vocab"], 6)
+    ref = plain("mixed", toks)
+    rows = [s.feed([("a", toks[:20], [19])])]
+    for t in range(20, 250):
+        rows.append(s.feed([("a", toks[t:t + 1], [0])]))
+    close_logits(torch.cat(rows), ref[19:], F32)
+
+
+def test_greedy_generation_through_the_scheduler():
+    cfg, w, model, s = build("mixed", F32, n_slots=2, max_step_tokens=16)
+    prompts = [tokens(9, cfg["vocab"], 31), tokens(21, cfg["vocab"], 32), tokens(3, cfg["vocab"], 33)]
+    outs = s.generate(prompts, 6)
+    for p, o in zip(prompts, outs):
+        seq = list(p)
+        for t in o:
+            lg = O.forward(cfg, w, seq)[-1]
+            top2 = torch.topk(lg, 2).values
+            if float(top2[0] - top2[1]) > 1e-3 * float(lg.abs().max()):     # a near tie may fall either way
+                assert int(torch.argmax(lg)) == t
+            seq.append(t)
+
+
+def test_checkpoint_folder_through_the_registry_the_command_line_and_the_trace_replay(tmp_path, capsys):
+    """config.json + model.safetensors -> registry -> the `generate` command and the replay program's main()."""
+    _cuda()
+    import io
+    import sys
+    import numpy as np
+    from qspec_b200 import registry
+    from qspec_b200.__main__ import main as cli
+    from qspec_b200.checkpoint import write_safetensors_file
+    from qspec_b200.legavik import LegavikConfig, random_weights
+    from qspec_b200.trace import main
+    cfg, rd, rg = CONFIGS["odd"]
+    w = random_weights(LegavikConfig.from_dict(cfg).with_ranks(decay_rank=rd, gate_rank=rg), 3)
+    with open(tmp_path / "config.json", "w") as f:
+        json.dump(cfg, f)
+    write_safetensors_file(str(tmp_path / "model.safetensors"), w)
+    assert type(registry.load_model(str(tmp_path), dtype="float32", n_slots=1, max_step_tokens=8, max_seq_tokens=32)).__name__ == "LegavikModel"
+    assert cli(["generate", "--model", str(tmp_path), "--dtype", "float32", "--prompt", "5,17,3", "--max-new-tokens", "2"]) == 0
+    line = json.loads(capsys.readouterr().out.strip().splitlines()[-1])
+    assert line["prompt"] == [5, 17, 3] and len(line["tokens"]) == 2
+    assert line["tokens"][0] == int(torch.argmax(O.forward(cfg, w, [5, 17, 3])[-1]))
+    toks = tokens(24, cfg["vocab"], 8)
+    steps = [{"step": 0, "entries": [{"id": "r", "tokens": toks[:11], "want": [0, 10]}], "end": []},
+             {"step": 1, "entries": [{"id": "r", "tokens": toks[11:13], "want": []}], "end": []},
+             {"step": 2, "entries": [{"id": "r", "tokens": toks[13:], "want": [10]}], "end": ["r"]},
+             {"step": 3, "entries": [{"id": "s", "tokens": toks[:2], "want": [1]}], "end": ["s"]}]
+    stdin, stdout = sys.stdin, sys.stdout
+    sys.stdin, sys.stdout = io.StringIO("\n".join(json.dumps(s) for s in steps) + "\n"), io.StringIO()
+    try:
+        rc = main(["--model", str(tmp_path), "--dtype", "float32", "--out", str(tmp_path / "out"), "--max-tokens", "32"])
+        printed = sys.stdout.getvalue()
+    finally:
+        sys.stdin, sys.stdout = stdin, stdout
+    assert rc == 0 and [l for l in printed.splitlines() if l.startswith("done")] == ["done 0", "done 1", "done 2", "done 3"]
+    ref = O.forward(cfg, w, toks)
+    assert not os.path.exists(tmp_path / "out" / "1.f32")
+    for step, rows in ((0, [0, 10]), (2, [23]), (3, [1])):
+        got = torch.from_numpy(np.fromfile(tmp_path / "out" / f"{step}.f32", dtype="<f4").reshape(len(rows), cfg["vocab"]))
+        close_logits(got, ref[rows], F32)
