@@ -111,7 +111,7 @@ head_prep_kernel(const qspec_head_prep_args a) {
   const int HD = H * D, GD = G * D, K1 = a.taps - 1, C = HD + GD + G * DV;
   const float* told = a.conv_w ? a.tail + ((size_t)mt.phase * a.slots + mt.slot) * K1 * C : nullptr;
   float* tnew = a.conv_w ? a.tail + ((size_t)(1 - mt.phase) * a.slots + mt.slot) * K1 * C : nullptr;
-  const bool last = i == mt.seg_end - 1;
+  const bool last = i == mt.seg_end - 1, inside = i - mt.seg_begin >= K1 && K1 < 4;
   const float temp = a.temp_every > 0 ? 1.0f + a.temp_coef * logf((float)((mt.pos + 1) / a.temp_every + 1)) : 1.0f;
   const size_t crow = (size_t)mt.slot * a.cap + (size_t)ring_row(mt.pos, a.keep_first, a.cap);
   const int NH = H + G + (a.v_off >= 0 ? G : 0);
@@ -128,6 +128,21 @@ head_prep_kernel(const qspec_head_prep_args a) {
       for (int e = 0; e < VEC; ++e) x[s].v[e] = 0.f;
       if (c >= n) continue;
       if (!a.conv_w) { x[s] = ldv<VEC>(prow + col + c); continue; }
+      if (inside) {                                               // (uniform over the warp) every tap lies in the step: loads without branches
+        VecF<VEC> u[4], wv[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const int back = min(j, K1);
+          u[j] = ldv<VEC>(prow - (size_t)back * a.ld + col + c);
+          wv[j] = ldv<VEC>(a.conv_w + (size_t)(K1 - back) * C + ch + c);
+        }
+#pragma unroll
+        for (int j = 3; j >= 0; --j)                              // oldest first, as below
+          if (j <= K1) {
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) x[s].v[e] += wv[j].v[e] * u[j].v[e];
+          }
+      } else
       for (int j = 0; j <= K1; ++j) {
         const int back = K1 - j, sp = mt.pos - back;              // source position
         VecF<VEC> u;
@@ -843,7 +858,7 @@ static int launch_head_prep(const qspec_head_prep_args& a, cudaStream_t st) {
   }
   // heads of a token go round grid y: enough CTAs to fill the GPU, few enough that a token's angles serve several heads
   const int nh = a.H + a.G + (a.v_off >= 0 ? a.G : 0), rows = (a.ntok + 7) / 8;
-  int gy = (148 * 8 + rows - 1) / rows;
+  int gy = (148 * 16 + rows - 1) / rows;
   if (gy > nh) gy = nh;
   if (gy > 65535) gy = 65535;
   launch_pdl(head_prep_kernel<T, VEC, NCV>, dim3(rows, gy), dim3(256), smem, st, a);
