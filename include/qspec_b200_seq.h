@@ -357,13 +357,16 @@ int qspec_seq_softcap_f32(float* a, long long n, float cap, void* stream);
  *   conv_w (float32 [taps][C], C = H D + G D + G DV channels in the order q, k, v; NULL: none): x_t <- sum_j conv_w[j] x_(t-taps+1+j),
  *     the rows before the step from tail (float32 [2][slots][taps - 1][C], read at `phase`, written at 1 - `phase`), zeros before
  *     position 0; values go to the cache as they are now
- *   norm_last 0: q, k <- x / sqrt(mean over D of x^2 + eps) * qn_w / kn_w (float32 [D], NULL: ones)
- *   rotation of the first rot_dims entries, entry i with entry i + rot_dims / 2 by the angle pos * inv_freq[i], cosine and sine
- *     times rot_amp
- *   norm_last 1: the norm comes here instead
+ *   norm_last QSPEC_HEAD_NORM_FIRST: q, k <- x / sqrt(mean over D of x^2 + eps) * qn_w / kn_w (float32 [D], NULL: ones)
+ *   rotation of the first rot_dims entries by the angles pos * inv_freq[i], paired as `pairing` says (QSPEC_ROTARY_*), cosine and
+ *     sine times rot_amp
+ *   norm_last QSPEC_HEAD_NORM_LAST: the norm comes here instead; QSPEC_HEAD_NORM_NONE: there is no norm
  *   temp_every > 0: q <- q * (1 + temp_coef * ln(floor((pos + 1) / temp_every) + 1))
  * qout float32 [ntok, H, D]; cache_k [slots, cap, G, D] and cache_v [slots, cap, G, DV] take ring row pos (keep_first as in
  * qspec_window_attn_args). D, DV <= 1024. */
+#define QSPEC_HEAD_NORM_FIRST 0
+#define QSPEC_HEAD_NORM_LAST  1
+#define QSPEC_HEAD_NORM_NONE  2
 typedef struct qspec_head_prep_args {
   const void* p; int ld, q_off, k_off, v_off;
   const float* conv_w; int taps; float* tail; int slots;
@@ -372,6 +375,7 @@ typedef struct qspec_head_prep_args {
   float temp_coef; int temp_every;
   float* qout; void* cache_k; void* cache_v; int cap, keep_first;
   const int* meta; int ntok, H, G, D, DV; float eps;
+  int pairing;
 } qspec_head_prep_args;
 int qspec_seq_head_prep(const qspec_head_prep_args* args, int dtype, void* stream);
 
@@ -400,6 +404,63 @@ typedef struct qspec_delta_channel_args {
 size_t qspec_seq_delta_channel_scratch_bytes(int nblocks, int ntok, int H, int D, int DV);
 int qspec_seq_delta_channel(const qspec_delta_channel_args* args, const int* block_rows, int nblocks, const int* long_starts,
                             const int* long_block0, int nlong, int max_len, void* scratch, size_t scratch_bytes, int dtype, void* stream);
+
+/* ---- matrix states with one decay per head and token, norms around the sublayer, gated norms in parts ---- */
+
+/* Residual sum between a norm of the sublayer's result and the norm of the next sublayer's input, in one launch:
+ *   v = sum_p y_w[t, p] * y[t, p, :] + y2[t, :]            (y_w NULL: ones; y2 NULL: no such term)
+ *   r = x_in + v / sqrt(mean(v^2) + eps) * (w_offset + post_w)      (y NULL: r = x_in)
+ *   out = r / sqrt(mean(r^2) + eps) * (w_offset + pre_w)
+ * r goes to x_out (float32, may alias x_in, may be NULL), the norm to out (activation type, may be NULL). y and y2 are of the
+ * activation type. W <= 16384. */
+int qspec_seq_sandwich_norm(const float* x_in, float* x_out, const void* y, int y_parts, long long y_part_stride,
+                            long long y_tok_stride, const float* y_w, const void* y2, const float* post_w, const float* pre_w,
+                            float w_offset, void* out, int ntok, int W, float eps, int dtype, void* stream);
+
+/* Norm of a row of N float32 entries in `parts` equal parts, each by its own root mean square, with a weight [N] and a gate:
+ *   SIGMOID_AFTER: out = out_scale * src / rms(src) * w * sigmoid(gate)
+ *   SILU_BEFORE:   u = src * silu(gate); out = out_scale * u / rms(u) * w */
+#define QSPEC_GATE_SIGMOID_AFTER 0
+#define QSPEC_GATE_SILU_BEFORE   1
+int qspec_seq_part_norm(const float* src, const float* w, const void* gate, int gate_ld, int gate_mode, void* out, int out_ld,
+                        int ntok, int N, int parts, float eps, float out_scale, int dtype, void* stream);
+
+/* Matrix state with one decay per head and token. Row t of p (leading dimension ld, activation type): q (G x D) at column q_off, k
+ * (G x D) at k_off, v (H x DV) at v_off; head h uses query / key head h / (H / G). Per head, S float32 [D, DV]:
+ *   S <- a_t S + dt_t k_t v_t^T;   y[t, h] = S^T q_t + D_skip[h] v_t          (D_skip NULL: no such term; y float32 [ntok, H, DV])
+ *   A_log NULL: a_t = decay[h], dt_t = 1 (log_decay[h] = ln decay[h]; float32, a large negative number for a decay of zero);
+ *   otherwise dt_t = softplus(dt[t, h] + dt_bias[h]) (dt of the activation type, leading dimension dt_ld), a_t = exp(-exp(A_log[h]) dt_t)
+ * q, k and v go through silu if `silu`; with conv_w (token form only) through a short causal convolution first: conv_w float32
+ * [conv_c, taps] (last column: the current token), conv_b float32 [conv_c] or NULL, channel = column - conv_off, tail float32 [2][slots]
+ * [taps - 1][conv_c] as for qspec_seq_conv_act. state: float32 [slots, H, D, DV], read at a segment's start (zero at position 0), written
+ * at its end. seg_starts int32 [nseg]: the first rows of all segments. D <= 256.
+ * _tokens: the segments of at most max_len tokens, token by token. _chunks: bfloat16, without convolution, the nlong segments whose first
+ * rows are `starts`; chunk_rows int32 [nchunks] holds the first row of every 64 tokens of those segments, in order, chunk0 int32 [nlong]
+ * the index in chunk_rows of a segment's first chunk. Section columns, ld, D and DV multiples of 8, p and state on 16-byte boundaries;
+ * scratch (bytes from the query) on 16-byte boundaries. */
+typedef struct qspec_scalar_decay_args {
+  const void* p; int ld, q_off, k_off, v_off, silu;
+  const float* conv_w; const float* conv_b; int taps, conv_off, conv_c; float* tail; int slots;
+  const float* decay; const float* log_decay;
+  const void* dt; int dt_ld; const float* dt_bias; const float* A_log;
+  const float* D_skip;
+  float* state; float* y;
+  const int* meta; const int* seg_starts; int nseg, ntok, H, G, D, DV;
+} qspec_scalar_decay_args;
+int qspec_seq_scalar_decay_tokens(const qspec_scalar_decay_args* args, int max_len, int dtype, void* stream);
+size_t qspec_seq_scalar_decay_scratch_bytes(int nchunks, int H, int D, int DV);
+int qspec_seq_scalar_decay_chunks_supported(int ld, int q_off, int k_off, int v_off, int D, int DV);
+int qspec_seq_scalar_decay_chunks(const qspec_scalar_decay_args* args, const int* chunk_rows, int nchunks, const int* starts,
+                                  const int* chunk0, int nlong, void* scratch, size_t scratch_bytes, void* stream);
+
+/* qspec_moe_route_chosen with a bias per output (float32 [R], NULL: none), part of the logits: z = router_w h + bias. */
+int qspec_moe_route_chosen_bias(const void* h, const float* router_w, const float* bias, int* idx, float* weight, int ntok, int W, int R,
+                                int top, int dtype, void* stream);
+
+/* out[t, f] = act(gu[t, f]) * gu[t, F + f]: rows of gu are [gate (F) | up (F)] with leading dimension ld; out [ntok, F]. */
+#define QSPEC_GLU_SILU      0
+#define QSPEC_GLU_GELU_TANH 1
+int qspec_seq_glu(const void* gu, int ld, void* out, int ntok, int F, int act, int dtype, void* stream);
 
 /* Arg max per row of float32 / bfloat16 logits [rows, V] (lowest index among equal maxima): int64 out. */
 int qspec_seq_argmax_rows(const void* logits, int rows, int V, long long row_stride, long long* out_idx, int dtype,

@@ -185,6 +185,16 @@ SEQ_SIGNATURES = {
     "qspec_seq_softcap_f32": (c_int, [c_void_p, c_ll, c_float, c_void_p]),
     "qspec_seq_head_prep": (c_int, [c_void_p, c_int, c_void_p]),
     "qspec_seq_delta_channel_scratch_bytes": (c_size_t, [c_int, c_int, c_int, c_int, c_int]),
+    "qspec_seq_sandwich_norm": (c_int, [c_void_p, c_void_p, c_void_p, c_int, c_ll, c_ll, c_void_p, c_void_p, c_void_p, c_void_p, c_float,
+                                        c_void_p, c_int, c_int, c_float, c_int, c_void_p]),
+    "qspec_seq_part_norm": (c_int, [c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float,
+                                    c_int, c_void_p]),
+    "qspec_seq_scalar_decay_tokens": (c_int, [c_void_p, c_int, c_int, c_void_p]),
+    "qspec_seq_scalar_decay_scratch_bytes": (c_size_t, [c_int, c_int, c_int, c_int]),
+    "qspec_seq_scalar_decay_chunks_supported": (c_int, [c_int, c_int, c_int, c_int, c_int, c_int]),
+    "qspec_seq_scalar_decay_chunks": (c_int, [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_size_t, c_void_p]),
+    "qspec_moe_route_chosen_bias": (c_int, [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p]),
+    "qspec_seq_glu": (c_int, [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p]),
     "qspec_seq_delta_channel": (c_int, [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_size_t, c_int, c_void_p]),
 }
 
@@ -209,7 +219,19 @@ class HeadPrepArgs(ctypes.Structure):
                 ("inv_freq", c_void_p), ("rot_dims", c_int), ("rot_amp", c_float),
                 ("temp_coef", c_float), ("temp_every", c_int),
                 ("qout", c_void_p), ("cache_k", c_void_p), ("cache_v", c_void_p), ("cap", c_int), ("keep_first", c_int),
-                ("meta", c_void_p), ("ntok", c_int), ("H", c_int), ("G", c_int), ("D", c_int), ("DV", c_int), ("eps", c_float)]
+                ("meta", c_void_p), ("ntok", c_int), ("H", c_int), ("G", c_int), ("D", c_int), ("DV", c_int), ("eps", c_float),
+                ("pairing", c_int)]
+
+
+class ScalarDecayArgs(ctypes.Structure):
+    """qspec_scalar_decay_args of include/qspec_b200_seq.h."""
+    _fields_ = [("p", c_void_p), ("ld", c_int), ("q_off", c_int), ("k_off", c_int), ("v_off", c_int), ("silu", c_int),
+                ("conv_w", c_void_p), ("conv_b", c_void_p), ("taps", c_int), ("conv_off", c_int), ("conv_c", c_int), ("tail", c_void_p),
+                ("slots", c_int), ("decay", c_void_p), ("log_decay", c_void_p),
+                ("dt", c_void_p), ("dt_ld", c_int), ("dt_bias", c_void_p), ("A_log", c_void_p), ("D_skip", c_void_p),
+                ("state", c_void_p), ("y", c_void_p),
+                ("meta", c_void_p), ("seg_starts", c_void_p), ("nseg", c_int), ("ntok", c_int), ("H", c_int), ("G", c_int), ("D", c_int),
+                ("DV", c_int)]
 
 
 class DeltaChannelArgs(ctypes.Structure):

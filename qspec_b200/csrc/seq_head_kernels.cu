@@ -60,33 +60,11 @@ template <int VEC> __global__ void __launch_bounds__(256) softcap_kernel(float* 
   }
 }
 
-// silu of a convolution's result: in bfloat16 mode (the inputs are bfloat16 roundings, relative 4e-3) the exponential and the
-// division run on the special-function unit
-template <typename T> __device__ __forceinline__ float silu_act(float z) { return silu_f(z); }
-template <> __device__ __forceinline__ float silu_act<bf16_t>(float z) { return __fdividef(z, 1.0f + __expf(-z)); }
-
-// ---- inputs of a short causal convolution -------------------------------------------------------------------------------------
-// The input of channel c at position sp: a row of the step, a row of the slot's tail (the last K1 inputs before the step), or zero
-// before the sequence's start.
-template <typename T> struct ConvRows {
-  const T* in;            // channel 0 of batch row seg_begin
-  int ld, first_pos, K1, C;
-  const float* told;      // [K1][C] of the slot, as it was before the step
-  __device__ __forceinline__ float get(int sp, int c) const {
-    if (sp >= first_pos) return to_f(in[(size_t)(sp - first_pos) * ld + c]);
-    return sp >= 0 ? told[(size_t)(sp - first_pos + K1) * C + c] : 0.f;
-  }
-  // the slot's new tail for channel c once the segment's last position is `last`
-  __device__ __forceinline__ void write_tail(float* tnew, int last, int c) const {
-    for (int r = 0; r < K1; ++r) tnew[(size_t)r * C + c] = get(last + 1 - K1 + r, c);
-  }
-};
-
 // ---- attention heads from the projection ----------------------------------------------------------------------------------------
 // One warp per token, eight consecutive tokens per CTA, the heads in turn (query heads, key heads, value heads); lanes hold VEC
 // neighbouring channels NCV times. Per head: convolution (optional), unit-RMS norm with a weight before the rotation or without
-// one after it, rotation of the first rot_dims entries (entry i with i + rot_dims / 2, angle pos * inv_freq[i], cosine and sine
-// times an amplitude), temperature of the queries. Values are a section of their own or the key heads as projected.
+// one after it or none, rotation of the first rot_dims entries (entry i with i + rot_dims / 2, or 2i with 2i + 1; angle pos *
+// inv_freq[i], cosine and sine times an amplitude), temperature of the queries. Values are a section of their own or the key heads as projected.
 template <typename T, int VEC, int NCV>
 __global__ void __launch_bounds__(256)
 head_prep_kernel(const qspec_head_prep_args a) {
@@ -191,8 +169,20 @@ head_prep_kernel(const qspec_head_prep_args a) {
         for (int e = 0; e < VEC; ++e) x[s].v[e] *= weight ? rr * weight[c + e] : rr;
       }
     };
-    if (!a.norm_last) unit(nw);
-    if (half) {
+    if (a.norm_last == QSPEC_HEAD_NORM_FIRST) unit(nw);
+    if (half && VEC == 4 && a.pairing == QSPEC_ROTARY_INTERLEAVED) {       // both entries of a pair lie in one lane
+#pragma unroll
+      for (int s = 0; s < NCV; ++s)
+#pragma unroll
+        for (int e = 0; e + 1 < VEC; e += 2) {
+          const int f = ((s * 32 + lane) * VEC + e) >> 1;
+          if (f < half) {
+            const float u = x[s].v[e], v = x[s].v[e + 1];
+            x[s].v[e] = u * s_cos[f] - v * s_sin[f];
+            x[s].v[e + 1] = v * s_cos[f] + u * s_sin[f];
+          }
+        }
+    } else if (half) {
 #pragma unroll
       for (int s = 0; s < NCV; ++s) {
         const int c = (s * 32 + lane) * VEC;
@@ -207,13 +197,18 @@ head_prep_kernel(const qspec_head_prep_args a) {
         for (int e = 0; e < VEC; ++e) {
           const int c = (s * 32 + lane) * VEC + e;
           if (c < 2 * half) {
+            if (a.pairing == QSPEC_ROTARY_INTERLEAVED) {
+              const int f = c >> 1;
+              x[s].v[e] = (c & 1) ? buf[c] * s_cos[f] + buf[c - 1] * s_sin[f] : buf[c] * s_cos[f] - buf[c + 1] * s_sin[f];
+              continue;
+            }
             const int f = c < half ? c : c - half;
             x[s].v[e] = c < half ? buf[c] * s_cos[f] - buf[c + half] * s_sin[f] : buf[c] * s_cos[f] + buf[c - half] * s_sin[f];
           }
         }
       __syncwarp();
     }
-    if (a.norm_last) unit(nw);
+    if (a.norm_last == QSPEC_HEAD_NORM_LAST) unit(nw);
     if (kind == 0) {
       float* qdst = a.qout + ((size_t)i * H + head) * D;
 #pragma unroll
@@ -895,6 +890,9 @@ extern "C" int qspec_seq_head_prep(const qspec_head_prep_args* a, int dtype, voi
                 QSPEC_ERR_INVALID_ARG, "seq_head_prep: sections outside the row (values taken from the keys need equal sizes and no convolution)");
   QSPEC_REQUIRE(!a->conv_w || (a->taps >= 1 && a->taps <= 64 && (a->tail || a->taps == 1) && a->slots > 0), QSPEC_ERR_INVALID_ARG,
                 "seq_head_prep: a convolution of %d taps", a->taps);
+  QSPEC_REQUIRE(a->norm_last >= QSPEC_HEAD_NORM_FIRST && a->norm_last <= QSPEC_HEAD_NORM_NONE &&
+                    (a->pairing == QSPEC_ROTARY_HALVES || a->pairing == QSPEC_ROTARY_INTERLEAVED), QSPEC_ERR_INVALID_ARG,
+                "seq_head_prep: norm %d, pairing %d", a->norm_last, a->pairing);
   HD_DTYPE_OK(dtype);
   if (a->ntok == 0) return QSPEC_OK;
   if (dtype == QSPEC_DTYPE_F32) return launch_head_prep_n<float>(*a, (cudaStream_t)stream);

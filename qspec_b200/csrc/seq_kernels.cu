@@ -597,6 +597,10 @@ route_kernel(const T* __restrict__ h, const float* __restrict__ rw, const float*
   if (warp != 0) return;
   if (chosen_only) {
     // the `top` largest logits, then a softmax over those alone (the first pick is their maximum)
+    if (corr) {                               // a bias that is part of the logits
+      for (int r = lane; r < R; r += 32) z[r] += corr[r];
+      __syncwarp();
+    }
     float first = 0.f, sum = 0.f;
     for (int k = 0; k < top; ++k) {
       float bv = -INFINITY;
@@ -1090,6 +1094,11 @@ extern "C" int qspec_moe_route(const void* h, const float* router_w, const float
 extern "C" int qspec_moe_route_chosen(const void* h, const float* router_w, int* idx, float* weight, int ntok, int W, int R, int top,
                                       int dtype, void* stream) {
   return route_any(h, router_w, nullptr, idx, weight, ntok, W, R, top, 1, dtype, stream);
+}
+
+extern "C" int qspec_moe_route_chosen_bias(const void* h, const float* router_w, const float* bias, int* idx, float* weight, int ntok, int W,
+                                           int R, int top, int dtype, void* stream) {
+  return route_any(h, router_w, bias, idx, weight, ntok, W, R, top, 1, dtype, stream);
 }
 
 extern "C" int qspec_moe_expert_tokens_act(const void* h, const void* gate_up, const void* down, const int* idx, void* out, int ntok, int W,

@@ -443,7 +443,7 @@ __global__ void __launch_bounds__(256) act_kernel(T* __restrict__ a, long long n
 }
 
 template <typename T, int VEC>
-__global__ void __launch_bounds__(256) silu_mul_kernel(const T* __restrict__ gu, int ld, T* __restrict__ out, int F, long long n) {
+__global__ void __launch_bounds__(256) glu_kernel(const T* __restrict__ gu, int ld, T* __restrict__ out, int F, long long n, int act) {
   pdl_enter();
   for (long long k = ((long long)blockIdx.x * 256 + threadIdx.x) * VEC; k < n; k += (long long)gridDim.x * 256 * VEC) {
     const long long t = k / F;
@@ -451,7 +451,12 @@ __global__ void __launch_bounds__(256) silu_mul_kernel(const T* __restrict__ gu,
     const VecF<VEC> g = ldv<VEC>(gu + (size_t)t * ld + f), u = ldv<VEC>(gu + (size_t)t * ld + F + f);
     VecF<VEC> o;
 #pragma unroll
-    for (int e = 0; e < VEC; ++e) o.v[e] = g.v[e] / (1.0f + expf(-g.v[e])) * u.v[e];
+    for (int e = 0; e < VEC; ++e) {
+      const float z = g.v[e];
+      // z sigmoid(z), or the tanh form of gelu: (1 + tanh u) / 2 = sigmoid(2 u)
+      const float s = act == QSPEC_GLU_GELU_TANH ? 1.5957691216057308f * (z + 0.044715f * z * z * z) : z;
+      o.v[e] = z / (1.0f + expf(-s)) * u.v[e];
+    }
     stv<VEC>(out + k, o);
   }
 }
@@ -901,8 +906,9 @@ extern "C" int qspec_seq_act(void* a, long long n, int act, int dtype, void* str
   return QSPEC_OK;
 }
 
-extern "C" int qspec_seq_silu_mul(const void* gu, int ld, void* out, int ntok, int F, int dtype, void* stream) {
-  QSPEC_REQUIRE(gu && out && ntok >= 0 && F > 0 && ld >= 2 * F, QSPEC_ERR_INVALID_ARG, "seq_silu_mul: bad arguments");
+extern "C" int qspec_seq_glu(const void* gu, int ld, void* out, int ntok, int F, int act, int dtype, void* stream) {
+  QSPEC_REQUIRE(gu && out && ntok >= 0 && F > 0 && ld >= 2 * F, QSPEC_ERR_INVALID_ARG, "seq_glu: bad arguments");
+  QSPEC_REQUIRE(act == QSPEC_GLU_SILU || act == QSPEC_GLU_GELU_TANH, QSPEC_ERR_INVALID_ARG, "seq_glu: unknown activation %d", act);
   MIX_DTYPE_OK(dtype);
   if (ntok == 0) return QSPEC_OK;
   const long long n = (long long)ntok * F;
@@ -912,14 +918,18 @@ extern "C" int qspec_seq_silu_mul(const void* gu, int ld, void* out, int ntok, i
   if (blocks > 148 * 16) blocks = 148 * 16;
   cudaStream_t st = (cudaStream_t)stream;
   if (dtype == QSPEC_DTYPE_F32) {
-    if (vec) launch_pdl(silu_mul_kernel<float, 4>, dim3((unsigned)blocks), dim3(256), 0, st, (const float*)gu, ld, (float*)out, F, n);
-    else launch_pdl(silu_mul_kernel<float, 1>, dim3((unsigned)blocks), dim3(256), 0, st, (const float*)gu, ld, (float*)out, F, n);
+    if (vec) launch_pdl(glu_kernel<float, 4>, dim3((unsigned)blocks), dim3(256), 0, st, (const float*)gu, ld, (float*)out, F, n, act);
+    else launch_pdl(glu_kernel<float, 1>, dim3((unsigned)blocks), dim3(256), 0, st, (const float*)gu, ld, (float*)out, F, n, act);
   } else {
-    if (vec) launch_pdl(silu_mul_kernel<bf16_t, 4>, dim3((unsigned)blocks), dim3(256), 0, st, (const bf16_t*)gu, ld, (bf16_t*)out, F, n);
-    else launch_pdl(silu_mul_kernel<bf16_t, 1>, dim3((unsigned)blocks), dim3(256), 0, st, (const bf16_t*)gu, ld, (bf16_t*)out, F, n);
+    if (vec) launch_pdl(glu_kernel<bf16_t, 4>, dim3((unsigned)blocks), dim3(256), 0, st, (const bf16_t*)gu, ld, (bf16_t*)out, F, n, act);
+    else launch_pdl(glu_kernel<bf16_t, 1>, dim3((unsigned)blocks), dim3(256), 0, st, (const bf16_t*)gu, ld, (bf16_t*)out, F, n, act);
   }
   QSPEC_CHECK_LAUNCH(1);
   return QSPEC_OK;
+}
+
+extern "C" int qspec_seq_silu_mul(const void* gu, int ld, void* out, int ntok, int F, int dtype, void* stream) {
+  return qspec_seq_glu(gu, ld, out, ntok, F, QSPEC_GLU_SILU, dtype, stream);
 }
 
 extern "C" int qspec_seq_lightning(const void* p, int ld, const float* decay, const float* norm_w, float* state, float* scratch, void* out,

@@ -9,29 +9,6 @@
 
 namespace qspec {
 
-__device__ __forceinline__ void tk_ldmatrix_x4(uint32_t (&r)[4], const __nv_bfloat16* p) {
-  const uint32_t a = (uint32_t)__cvta_generic_to_shared(p);
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];\n" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
-}
-__device__ __forceinline__ void tk_ldmatrix_x4_trans(uint32_t (&r)[4], const __nv_bfloat16* p) {
-  const uint32_t a = (uint32_t)__cvta_generic_to_shared(p);
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];\n" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
-}
-// (hi, lo) split of two float32 weights: hi = bf16(w), lo = bf16(w - hi); hi + lo carries 16 mantissa bits
-__device__ __forceinline__ void tk_split_bf2(float w0, float w1, uint32_t& hi, uint32_t& lo) {
-  const __nv_bfloat16 h0 = __float2bfloat16_rn(w0), h1 = __float2bfloat16_rn(w1);
-  __nv_bfloat162 hv, lv;
-  hv.x = h0; hv.y = h1;
-  lv = __floats2bfloat162_rn(w0 - __bfloat162float(h0), w1 - __bfloat162float(h1));
-  hi = *reinterpret_cast<uint32_t*>(&hv);
-  lo = *reinterpret_cast<uint32_t*>(&lv);
-}
-__device__ __forceinline__ void tk_mma_16816(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
-               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-
 // ---- short causal convolution over time, per channel, with an activation ---------------------------------------------------
 // out[t, c] = act(bias[c] + sum_j w[c, j] * in[t - taps + 1 + j, c]). Rows before the segment's first token come from the
 // slot's tail (the last taps - 1 inputs of the sequence so far), rows before position 0 are zero. One thread per (token,
@@ -80,6 +57,66 @@ conv_act_kernel(const T* __restrict__ in, int ld, const float* __restrict__ w, c
       if (sp >= first_pos) v = to_f(in[(size_t)(mt.seg_begin + sp - first_pos) * ld + c]);
       else if (sp >= 0) v = told[(size_t)(sp - (first_pos - K1)) * C + c];
       tnew[(size_t)r * C + c] = v;
+    }
+  }
+}
+
+// The same for filters of at most KT taps over channels in groups of four: a thread owns four neighbouring channels of RUN
+// consecutive batch rows, keeps the last KT - 1 inputs and its weights in registers and loads every row once, all of them before the
+// first is used. Rows in front of the run come from the step (same segment), from the tail, or are zero. Sums in the order of
+// conv_act_kernel.
+template <typename T, typename OT, int KT, int RUN>
+__global__ void __launch_bounds__(256)
+conv_act_run_kernel(const T* __restrict__ in, int ld, const float* __restrict__ w, const float* __restrict__ bias, int taps,
+                    float* __restrict__ tail, int slots, OT* __restrict__ out, int out_ld, const int* __restrict__ meta, int ntok, int C,
+                    int act) {
+  pdl_enter();
+  const int i0 = blockIdx.x * RUN, c = (blockIdx.y * 256 + threadIdx.x) * 4;
+  if (c >= C) return;
+  const int K1 = taps - 1;
+  VecF<4> rows[RUN], hist[KT], wv[KT], b;
+#pragma unroll
+  for (int r = 0; r < RUN; ++r) rows[r] = ldv<4>(in + (size_t)min(i0 + r, ntok - 1) * ld + c);
+#pragma unroll
+  for (int j = 0; j < KT; ++j)                                    // leading weights of a shorter filter are zero
+#pragma unroll
+    for (int e = 0; e < 4; ++e) wv[j].v[e] = j >= KT - taps ? w[(size_t)(c + e) * taps + j - (KT - taps)] : 0.f;
+#pragma unroll
+  for (int e = 0; e < 4; ++e) b.v[e] = bias ? bias[c + e] : 0.f;
+  // input of the sequence of `mt` at position sp (before the segment's token `i`, or in it)
+  auto get = [&](const TokMeta& mt, int first_pos, int sp) {
+    VecF<4> v;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) v.v[e] = 0.f;
+    if (sp >= first_pos) v = ldv<4>(in + (size_t)(mt.seg_begin + sp - first_pos) * ld + c);
+    else if (sp >= 0 && sp >= first_pos - K1) v = ldv<4>(tail + (((size_t)mt.phase * slots + mt.slot) * K1 + (sp - first_pos + K1)) * C + c);
+    return v;
+  };
+#pragma unroll
+  for (int r = 0; r < RUN; ++r) {
+    const int i = i0 + r;
+    if (i < ntok) {
+      const TokMeta mt = load_meta(meta, ntok, i);
+      const int first_pos = mt.pos - (i - mt.seg_begin);
+      if (r == 0 || i == mt.seg_begin) {
+#pragma unroll
+        for (int j = 0; j < KT - 1; ++j) hist[j] = get(mt, first_pos, mt.pos - (KT - 1) + j);
+      }
+      hist[KT - 1] = rows[r];
+      VecF<4> acc = b;
+#pragma unroll
+      for (int j = 0; j < KT; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc.v[e] += wv[j].v[e] * hist[j].v[e];
+      if (act == QSPEC_CONV_ACT_SILU)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc.v[e] = silu_f(acc.v[e]);
+      stv<4>(out + (size_t)i * out_ld + c, acc);
+      if (i == mt.seg_end - 1)
+        for (int k = 0; k < K1; ++k)
+          stv<4>(tail + (((size_t)(1 - mt.phase) * slots + mt.slot) * K1 + k) * C + c, get(mt, first_pos, mt.pos + 1 - K1 + k));
+#pragma unroll
+      for (int j = 0; j < KT - 1; ++j) hist[j] = hist[j + 1];
     }
   }
 }
@@ -877,6 +914,29 @@ extern "C" int qspec_seq_conv_act(const void* in, int ld, const float* w, const 
   if (ntok == 0) return QSPEC_OK;
   const dim3 grid(ntok, (C + 255) / 256);
   cudaStream_t st = (cudaStream_t)stream;
+  // groups of four channels whose rows start on group boundaries, short filters: runs of rows per thread
+  const size_t es = dtype == QSPEC_DTYPE_F32 ? 4 : 2, oes = (dtype == QSPEC_DTYPE_F32 || out_f32) ? 4 : 2;
+  const bool runs = taps <= 4 && C % 4 == 0 && ld % 4 == 0 && out_ld % 4 == 0 && ((uintptr_t)in & (4 * es - 1)) == 0 &&
+                    ((uintptr_t)out & (4 * oes - 1)) == 0 && ((uintptr_t)tail & 15) == 0;
+  if (runs) {
+    // long runs once they fill the GPU, single rows below
+    const int groups = (C + 1023) / 1024;
+    const bool eight = (long long)(ntok / 8) * groups >= 296;
+    const dim3 rgrid(eight ? (ntok + 7) / 8 : ntok, groups);
+#define CR_ARGS(T, OT) (const T*)in, ld, w, bias, taps, tail, slots, (OT*)out, out_ld, meta, ntok, C, act
+#define CR_LAUNCH(T, OT)                                                                                                       \
+  do {                                                                                                                         \
+    if (eight) launch_pdl(conv_act_run_kernel<T, OT, 4, 8>, rgrid, dim3(256), 0, st, CR_ARGS(T, OT));                          \
+    else launch_pdl(conv_act_run_kernel<T, OT, 4, 1>, rgrid, dim3(256), 0, st, CR_ARGS(T, OT));                                \
+  } while (0)
+    if (dtype == QSPEC_DTYPE_F32) CR_LAUNCH(float, float);
+    else if (out_f32) CR_LAUNCH(bf16_t, float);
+    else CR_LAUNCH(bf16_t, bf16_t);
+#undef CR_LAUNCH
+#undef CR_ARGS
+    QSPEC_CHECK_LAUNCH(1);
+    return QSPEC_OK;
+  }
 #define CV_ARGS w, bias, taps, tail, slots
   if (dtype == QSPEC_DTYPE_F32)
     launch_pdl(conv_act_kernel<float, float>, grid, dim3(256), 0, st, (const float*)in, ld, CV_ARGS, (float*)out, out_ld, meta, ntok, C, act);

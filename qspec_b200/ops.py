@@ -918,15 +918,19 @@ def moe_expert_grouped(h: torch.Tensor, gate_up: Optional[torch.Tensor], down: O
                                           EXPERT_ACTS[act], _ptr(ws), ws.numel(), _stream()), "moe_expert_grouped")
 
 
-def moe_route_chosen(h: torch.Tensor, router_w: torch.Tensor, idx: torch.Tensor, weight: torch.Tensor) -> None:
-    """Router whose weights are a softmax over the chosen logits only: the `top` largest of router_w h (float32)."""
+def moe_route_chosen(h: torch.Tensor, router_w: torch.Tensor, idx: torch.Tensor, weight: torch.Tensor,
+                     bias: Optional[torch.Tensor] = None) -> None:
+    """Router whose weights are a softmax over the chosen logits only: the `top` largest of router_w h (+ bias, float32 [R])."""
+    _chk(bias, "bias", (_F32,), allow_none=True)
     _chk(h, "h", _SEQ_ACT); _chk(router_w, "router_w", (_F32,)); _chk(idx, "idx", (torch.int32,)); _chk(weight, "weight", (_F32,))
     ntok, W = h.shape
     R, top = router_w.shape[0], idx.shape[1]
     if router_w.shape[1] != W or idx.shape != (ntok, top) or weight.shape != (ntok, top):
         raise ValueError("moe_route_chosen: shapes do not match")
-    _seq(_lib.load_seq().qspec_moe_route_chosen(_ptr(h), _ptr(router_w), _ptr(idx), _ptr(weight), ntok, W, R, top, _sdt(h), _stream()),
-         "moe_route_chosen")
+    if bias is not None and bias.numel() != R:
+        raise ValueError("moe_route_chosen: one bias per router output")
+    _seq(_lib.load_seq().qspec_moe_route_chosen_bias(_ptr(h), _ptr(router_w), _ptr(bias), _ptr(idx), _ptr(weight), ntok, W, R, top, _sdt(h),
+                                                     _stream()), "moe_route_chosen")
 
 
 def seq_token_shift(x: torch.Tensor, shift: torch.Tensor, prev: torch.Tensor, out: torch.Tensor, meta: torch.Tensor) -> None:
@@ -1169,13 +1173,21 @@ def seq_act(a: torch.Tensor, act: str) -> None:
     _seq(_lib.load_seq().qspec_seq_act(_ptr(a), a.numel(), SEQ_ACTS[act], _sdt(a), _stream()), "seq_act")
 
 
-def seq_silu_mul(gu: torch.Tensor, out: torch.Tensor) -> None:
-    """out [ntok, F] = silu(gu[:, :F]) * gu[:, F:] for rows [gate | up]."""
+GLU_ACTS = {"silu": 0, "gelu_tanh": 1}
+
+
+def seq_glu(gu: torch.Tensor, out: torch.Tensor, act: str) -> None:
+    """out [ntok, F] = act(gu[:, :F]) * gu[:, F:] for rows [gate | up]; act "silu" or "gelu_tanh"."""
     _chk(gu, "gu", _SEQ_ACT); _chk(out, "out", (gu.dtype,))
     ntok, F = out.shape
     if gu.shape != (ntok, 2 * F):
-        raise ValueError("seq_silu_mul: gu must be [ntok, 2 F]")
-    _seq(_lib.load_seq().qspec_seq_silu_mul(_ptr(gu), 2 * F, _ptr(out), ntok, F, _sdt(gu), _stream()), "seq_silu_mul")
+        raise ValueError("seq_glu: gu must be [ntok, 2 F]")
+    _seq(_lib.load_seq().qspec_seq_glu(_ptr(gu), 2 * F, _ptr(out), ntok, F, GLU_ACTS[act], _sdt(gu), _stream()), "seq_glu")
+
+
+def seq_silu_mul(gu: torch.Tensor, out: torch.Tensor) -> None:
+    """out [ntok, F] = silu(gu[:, :F]) * gu[:, F:] for rows [gate | up]."""
+    seq_glu(gu, out, "silu")
 
 
 def seq_lightning(p: torch.Tensor, decay: torch.Tensor, norm_w: torch.Tensor, state: torch.Tensor, scratch: torch.Tensor,
@@ -1444,11 +1456,12 @@ def seq_head_prep(p: torch.Tensor, q_off: int, k_off: int, v_off: Optional[int],
                   cache_v: torch.Tensor, meta: torch.Tensor, H: int, eps: float, *, conv_w: Optional[torch.Tensor] = None,
                   tail: Optional[torch.Tensor] = None, qn_w: Optional[torch.Tensor] = None, kn_w: Optional[torch.Tensor] = None,
                   norm_last: bool = False, inv_freq: Optional[torch.Tensor] = None, rot_dims: int = 0, rot_amp: float = 1.0,
-                  temp_coef: float = 0.0, temp_every: int = 0, keep_first: int = 0) -> None:
+                  temp_coef: float = 0.0, temp_every: int = 0, keep_first: int = 0, norm: bool = True, pairing: str = "halves") -> None:
     """Attention heads from the projection rows p [ntok, ld] (q [H x D], k [G x D], v [G x DV] at the given columns; v_off None: the
     values are the keys as projected): short convolution over q, k, v (conv_w float32 [taps, H D + G D + G DV], the last row meets the
     current token; tail float32 [2, slots, taps - 1, channels]), unit-RMS norm per head with the weights qn_w / kn_w (None: ones) before
-    the rotation -- after it if norm_last --, rotation of the first rot_dims entries by pos * inv_freq with the amplitude rot_amp, and
+    the rotation -- after it if norm_last, nowhere if not norm --, rotation of the first rot_dims entries by pos * inv_freq (pairing
+    "halves" or "interleaved") with the amplitude rot_amp, and
     q * (1 + temp_coef ln(floor((pos + 1) / temp_every) + 1)) if temp_every > 0. qout float32 [ntok, H, D]; cache_k [slots, cap, G, D]
     and cache_v [slots, cap, G, DV] of p's type take ring row pos, the first keep_first rows never reused."""
     import ctypes
@@ -1468,9 +1481,9 @@ def seq_head_prep(p: torch.Tensor, q_off: int, k_off: int, v_off: Optional[int],
         if conv_w.shape != (taps, C) or tail.shape != (2, slots, taps - 1, C):
             raise ValueError("seq_head_prep: the convolution and its tail have H D + G D + G DV channels")
     a = _lib.HeadPrepArgs(p.data_ptr(), p.stride(0), int(q_off), int(k_off), -1 if v_off is None else int(v_off), _ptr(conv_w), taps,
-                          _ptr(tail), slots, _ptr(qn_w), _ptr(kn_w), int(norm_last), _ptr(inv_freq), int(rot_dims), float(rot_amp),
+                          _ptr(tail), slots, _ptr(qn_w), _ptr(kn_w), (1 if norm_last else 0) if norm else 2, _ptr(inv_freq), int(rot_dims), float(rot_amp),
                           float(temp_coef), int(temp_every), _ptr(qout), _ptr(cache_k), _ptr(cache_v), cap, int(keep_first), _ptr(meta),
-                          ntok, H, G, D, DV, float(eps))
+                          ntok, H, G, D, DV, float(eps), ROTARY_PAIRINGS[pairing])
     _seq(_lib.load_seq().qspec_seq_head_prep(ctypes.byref(a), _sdt(p), _stream()), "seq_head_prep")
 
 
@@ -1515,3 +1528,118 @@ def seq_delta_channel(p: torch.Tensor, beta_off: int, conv_w: torch.Tensor, tail
                                                  scratch.data_ptr() if scratch is not None else None,
                                                  scratch.numel() * scratch.element_size() if scratch is not None else 0, _sdt(p), _stream()),
          "seq_delta_channel")
+
+
+# ---- matrix states with one decay per head and token, norms around the sublayer, gated norms in parts ---------------------------------
+
+def seq_sandwich_norm(x_in: torch.Tensor, eps: float, *, y: Optional[torch.Tensor] = None, y_w: Optional[torch.Tensor] = None,
+                      y2: Optional[torch.Tensor] = None, post_w: Optional[torch.Tensor] = None, pre_w: Optional[torch.Tensor] = None,
+                      x_out: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None, w_offset: float = 1.0) -> None:
+    """r = x_in + unit_rms(v) * (w_offset + post_w) with v = sum_p y_w[t, p] y[t, p] + y2 (y [ntok, W] or [ntok, parts, W]; no y: r =
+    x_in); out = unit_rms(r) * (w_offset + pre_w). x_in, x_out (may be x_in) float32 [ntok, W]; y, y2, out of the activation type."""
+    _chk(x_in, "x_in", (_F32,)); _chk(x_out, "x_out", (_F32,), allow_none=True); _chk(out, "out", _SEQ_ACT, allow_none=True)
+    for t, n in ((y_w, "y_w"), (post_w, "post_w"), (pre_w, "pre_w")):
+        _chk(t, n, (_F32,), allow_none=True)
+    ntok, W = x_in.shape
+    act = next((t for t in (out, y) if t is not None), x_in)
+    parts = y.shape[1] if y is not None and y.dim() == 3 else 1
+    for t, n in ((y, "y"), (y2, "y2")):
+        _chk(t, n, (act.dtype,), allow_none=True)
+    if (y is not None and (y.numel() != ntok * parts * W or y.shape[0] != ntok)) or (y_w is not None and y_w.shape != (ntok, parts)) or \
+            any(t is not None and t.shape != (ntok, W) for t in (y2, x_out, out)) or \
+            any(t is not None and t.numel() != W for t in (post_w, pre_w)):
+        raise ValueError("seq_sandwich_norm: shapes do not match")
+    _seq(_lib.load_seq().qspec_seq_sandwich_norm(_ptr(x_in), _ptr(x_out), _ptr(y), parts, W, parts * W, _ptr(y_w), _ptr(y2), _ptr(post_w),
+                                                 _ptr(pre_w), float(w_offset), _ptr(out), ntok, W, float(eps), _sdt(act), _stream()),
+         "seq_sandwich_norm")
+
+
+GATE_MODES = {"sigmoid_after": 0, "silu_before": 1}
+
+
+def seq_part_norm(src: torch.Tensor, w: torch.Tensor, gate: torch.Tensor, gate_mode: str, out: torch.Tensor, eps: float, parts: int = 1,
+                  out_scale: float = 1.0) -> None:
+    """Norm of rows src float32 [ntok, N] in `parts` equal parts with a weight [N] and a gate (view of the activation type, [ntok, N]):
+    "sigmoid_after": out = out_scale * unit_rms(src) * w * sigmoid(gate); "silu_before": out = out_scale * unit_rms(src * silu(gate)) * w."""
+    _chk(src, "src", (_F32,)); _chk(w, "w", (_F32,)); _rows(gate, "gate", _SEQ_ACT); _rows(out, "out", (gate.dtype,))
+    ntok, N = src.shape
+    if gate.shape != (ntok, N) or out.shape != (ntok, N) or w.numel() != N or parts < 1 or N % parts:
+        raise ValueError("seq_part_norm: shapes do not match")
+    _seq(_lib.load_seq().qspec_seq_part_norm(_ptr(src), _ptr(w), gate.data_ptr(), gate.stride(0), GATE_MODES[gate_mode], out.data_ptr(),
+                                             out.stride(0), ntok, N, int(parts), float(eps), float(out_scale), _sdt(gate), _stream()),
+         "seq_part_norm")
+
+
+def seq_scalar_decay_scratch_bytes(nchunks: int, H: int, D: int, DV: int) -> int:
+    """Bytes of scratch that `seq_scalar_decay` needs for nchunks chunks of 64 tokens."""
+    return int(_lib.load_seq().qspec_seq_scalar_decay_scratch_bytes(int(nchunks), H, D, DV))
+
+
+def seq_scalar_decay_chunks_supported(p: torch.Tensor, q_off: int, k_off: int, v_off: int, D: int, DV: int) -> bool:
+    """Whether the 64-token tensor-core form takes these sections of the rows p (bfloat16)."""
+    return p.dtype == _BF16 and p.data_ptr() % 16 == 0 and \
+        bool(_lib.load_seq().qspec_seq_scalar_decay_chunks_supported(p.stride(0), q_off, k_off, v_off, D, DV))
+
+
+def seq_scalar_decay(p: torch.Tensor, q_off: int, k_off: int, v_off: int, G: int, state: torch.Tensor, y: torch.Tensor, meta, *,
+                     silu: bool = True, decay: Optional[torch.Tensor] = None, log_decay: Optional[torch.Tensor] = None,
+                     dt: Optional[torch.Tensor] = None, dt_bias: Optional[torch.Tensor] = None, A_log: Optional[torch.Tensor] = None,
+                     D_skip: Optional[torch.Tensor] = None, conv: Optional[tuple] = None, conv_out: Optional[torch.Tensor] = None,
+                     scratch: Optional[torch.Tensor] = None) -> None:
+    """Matrix state with one decay per head and token: S <- a_t S + dt_t k_t v_t^T, y_t = S^T q_t (+ D_skip v_t), state float32 [slots, H,
+    D, DV], y float32 [ntok, H * DV]. Rows p hold q (G x D), k (G x D) and v (H x DV) at the given columns, through silu if `silu`. Fixed
+    decays (decay and log_decay = ln decay, float32 [H]), or dt_t = softplus(dt + dt_bias), a_t = exp(-exp(A_log) dt_t) with dt [ntok, H] a
+    view of p's type. conv = (weights float32 [channels, taps], bias or None, first column, tail float32 [2, slots, taps - 1, channels]): a
+    short causal convolution in front of the silu over these columns of p, which must include the three sections.
+
+    meta: the step's `state.BatchMeta`. Without scratch (uint8) every segment goes token by token. With it, segments of more than CHUNK_MIN
+    tokens take the 64-token form where the sizes allow (bfloat16); a convolution then runs as a launch of its own over the whole step, into
+    conv_out [ntok, channels] (view), which both forms read."""
+    import ctypes
+    from .state import CHUNK_MIN
+    _rows(p, "p", _SEQ_ACT); _chk(state, "state", (_F32,)); _chk(y, "y", (_F32,))
+    for t, n in ((decay, "decay"), (log_decay, "log_decay"), (dt_bias, "dt_bias"), (A_log, "A_log"), (D_skip, "D_skip")):
+        _chk(t, n, (_F32,), allow_none=True)
+    ntok = p.shape[0]
+    slots, H, D, DV = state.shape
+    if y.shape != (ntok, H * DV) or meta.table.shape != (5, ntok) or any(t is not None and t.numel() != H for t in
+                                                                         (decay, log_decay, dt_bias, A_log, D_skip)):
+        raise ValueError("seq_scalar_decay: shapes do not match")
+    if (A_log is None) != (decay is not None and log_decay is not None) or (A_log is not None and (dt is None or dt_bias is None)):
+        raise ValueError("seq_scalar_decay: either decay and log_decay, or dt, dt_bias and A_log")
+    if dt is not None:
+        _rows(dt, "dt", (p.dtype,))
+        if dt.shape != (ntok, H):
+            raise ValueError("seq_scalar_decay: one step size per token and head")
+    nlong, nchunks = meta.chunk_starts.numel(), meta.chunk_rows.numel()
+    cw, cb, c0, tail = conv if conv is not None else (None, None, 0, None)
+    if cw is not None:
+        _chk(cw, "conv weights", (_F32,)); _chk(cb, "conv bias", (_F32,), allow_none=True); _chk(tail, "tail", (_F32,))
+        C, taps = cw.shape
+        if not 0 <= c0 <= p.shape[1] - C or tail.shape != (2, slots, taps - 1, C) or (cb is not None and cb.numel() != C):
+            raise ValueError("seq_scalar_decay: the convolution and its tail do not match")
+    src, off = (conv_out, c0) if cw is not None else (p, 0)
+    chunks = nlong > 0 and scratch is not None and src is not None and \
+        seq_scalar_decay_chunks_supported(src, q_off - off, k_off - off, v_off - off, D, DV)
+
+    def args(rows, shift, act, with_conv):
+        return _lib.ScalarDecayArgs(rows.data_ptr(), rows.stride(0), int(q_off - shift), int(k_off - shift), int(v_off - shift), int(act),
+                                    _ptr(cw) if with_conv else None, _ptr(cb) if with_conv else None, cw.shape[1] if with_conv else 0,
+                                    int(c0) if with_conv else 0, cw.shape[0] if with_conv else 0, _ptr(tail) if with_conv else None, slots,
+                                    _ptr(decay), _ptr(log_decay), dt.data_ptr() if dt is not None else None,
+                                    dt.stride(0) if dt is not None else 0, _ptr(dt_bias), _ptr(A_log), _ptr(D_skip), _ptr(state), _ptr(y),
+                                    _ptr(meta.table), _ptr(meta.seg_starts), meta.seg_starts.numel(), ntok, H, int(G), D, DV)
+
+    lib = _lib.load_seq()
+    if not chunks:
+        a = args(p, 0, silu, cw is not None)
+        _seq(lib.qspec_seq_scalar_decay_tokens(ctypes.byref(a), 1 << 30, _sdt(p), _stream()), "seq_scalar_decay")
+        return
+    if cw is not None:
+        seq_conv_act(p[:, c0:c0 + cw.shape[0]], cw, cb, tail, conv_out, meta.table, act="silu" if silu else None)
+    a = args(src, off, silu and cw is None, False)
+    _seq(lib.qspec_seq_scalar_decay_chunks(ctypes.byref(a), meta.chunk_rows.data_ptr(), nchunks, meta.chunk_starts.data_ptr(),
+                                           meta.chunk_first.data_ptr(), nlong, scratch.data_ptr(), scratch.numel() * scratch.element_size(),
+                                           _stream()), "seq_scalar_decay")
+    if nlong < len(meta.segments):
+        _seq(lib.qspec_seq_scalar_decay_tokens(ctypes.byref(a), CHUNK_MIN, _sdt(p), _stream()), "seq_scalar_decay")

@@ -21,6 +21,8 @@ import torch
 META_ROWS = 5          # slot, pos, seg_begin, seg_end, phase (include/qspec_b200_seq.h)
 SCAN_BLOCK = 16        # tokens per block of the recurrences that are evaluated block by block
 SCAN_SHORT = 8         # segments of at most this many tokens go token by token instead
+CHUNK = 64             # tokens per chunk of the recurrences that run on the tensor cores
+CHUNK_MIN = 32         # segments of at most this many tokens go token by token instead
 
 
 class SlotPool:
@@ -59,6 +61,9 @@ class BatchMeta:
     block_rows: torch.Tensor                           # device int32: first row of every SCAN_BLOCK tokens of the segments longer than SCAN_SHORT
     long_starts: torch.Tensor                          # device int32: first row of every such segment
     long_block0: torch.Tensor                          # device int32: where such a segment's blocks begin in block_rows
+    chunk_rows: torch.Tensor                           # device int32: the same for CHUNK tokens of the segments longer than CHUNK_MIN ...
+    chunk_starts: torch.Tensor
+    chunk_first: torch.Tensor
 
     @property
     def max_length(self) -> int:
@@ -126,7 +131,7 @@ class SequenceTable:
         if len(set(slots)) != len(slots):
             raise ValueError("a request appears twice in one step")
         begin = np.cumsum(counts) - counts
-        h = np.zeros((META_ROWS + 6, ntok), dtype=np.int32)
+        h = np.zeros((META_ROWS + 9, ntok), dtype=np.int32)
         h[0] = np.repeat(np.asarray(slots, dtype=np.int64), counts)
         h[2] = np.repeat(begin, counts)
         h[1] = np.repeat(np.asarray(firsts, dtype=np.int64), counts) + (np.arange(ntok) - h[2])
@@ -139,21 +144,31 @@ class SequenceTable:
             nrows = len(rows)
             h[META_ROWS + 1, :nrows] = np.asarray(rows, dtype=np.int64)
         h[META_ROWS + 2, :len(counts)] = begin         # one entry per segment (a segment has at least one token)
-        long = counts > SCAN_SHORT
-        per = -(-counts[long] // SCAN_BLOCK)
-        nblk, nlong = int(per.sum()), int(long.sum())
-        if nlong:
-            first = np.cumsum(per) - per
-            h[META_ROWS + 3, :nblk] = np.repeat(begin[long], per) + SCAN_BLOCK * (np.arange(nblk) - np.repeat(first, per))
-            h[META_ROWS + 4, :nlong] = begin[long]
-            h[META_ROWS + 5, :nlong] = first
+
+        def blocks(row, size, longer_than):
+            """Rows row .. row + 2: first batch row of every `size` tokens of the long segments, the segments' first rows, the index of
+            their first block. Returns the number of blocks and of such segments."""
+            long = counts > longer_than
+            per = -(-counts[long] // size)
+            nblk, nlong = int(per.sum()), int(long.sum())
+            if nlong:
+                first = np.cumsum(per) - per
+                h[row, :nblk] = np.repeat(begin[long], per) + size * (np.arange(nblk) - np.repeat(first, per))
+                h[row + 1, :nlong] = begin[long]
+                h[row + 2, :nlong] = first
+            return nblk, nlong
+
+        nblk, nlong = blocks(META_ROWS + 3, SCAN_BLOCK, SCAN_SHORT)
+        nchunk, nlong64 = blocks(META_ROWS + 6, CHUNK, CHUNK_MIN)
         t = torch.from_numpy(h)
         if self.device.type == "cuda":
             t = t.pin_memory()
         dev = t.to(self.device, non_blocking=True)
         return BatchMeta(table=dev[:META_ROWS], ids=dev[META_ROWS], rows=dev[META_ROWS + 1, :nrows],
                          seg_starts=dev[META_ROWS + 2, :len(segs)], ntok=ntok, segments=segs, block_rows=dev[META_ROWS + 3, :nblk],
-                         long_starts=dev[META_ROWS + 4, :nlong], long_block0=dev[META_ROWS + 5, :nlong])
+                         long_starts=dev[META_ROWS + 4, :nlong], long_block0=dev[META_ROWS + 5, :nlong],
+                         chunk_rows=dev[META_ROWS + 6, :nchunk], chunk_starts=dev[META_ROWS + 7, :nlong64],
+                         chunk_first=dev[META_ROWS + 8, :nlong64])
 
     def commit(self, meta: BatchMeta) -> None:
         """The step described by `meta` has been queued: its tokens now count as consumed."""
