@@ -40,6 +40,7 @@ from typing import Dict, List, Optional
 import torch
 
 from . import ops
+from .seq_layers import PROMPT_TILES_MIN_CTAS, TILES_MIN_TOKENS, attend_window, run_experts
 from .state import SCAN_SHORT, BatchMeta
 
 UNIT_EPS = 1e-6                     # under the root of the delta rule's unit vectors
@@ -425,8 +426,7 @@ class LegavikModel(torch.nn.Module):
         self.buf_pair = torch.empty(T * tops * W if ffs else 1, **act)
         # bfloat16 takes the tensor-core forms where the sizes allow (as in repepel.RepepelModel); QSPEC_SEQ_TILES=0 keeps the plain ones
         self.use_tiles = dtype == torch.bfloat16 and os.environ.get("QSPEC_SEQ_TILES", "1") != "0"
-        self.tiles_min_tokens = 64           # a step with fewer tokens, or fewer than 16 per sequence, is decode-shaped
-        self.prompt_tiles_min_ctas = 64      # (64-token blocks x heads) from which a prompt portion takes the tile form of its attention
+        self.tiles_min_tokens, self.prompt_tiles_min_ctas = TILES_MIN_TOKENS, PROMPT_TILES_MIN_CTAS
         self._mm_f32_out = None              # whether torch.mm takes bfloat16 operands with a float32 out (probed once)
 
     # ------------------------------------------------------------------------------------------
@@ -465,21 +465,9 @@ class LegavikModel(torch.nn.Module):
     # ------------------------------------------------------------------------------------------
     def _attend(self, i, a: LegavikAttention, qf, gate, out, out_scale, meta: BatchMeta, T):
         """Softmax attention of the step's queries over the layer's cache rows, one sigmoid gate per head, into `out` [T, H, DV]."""
-        ck, cv = self.cache_k[i], self.cache_v[i]
-        window = a.window or FULL_WINDOW
-        kw = dict(gate=gate, gate_per_head=True, keep_first=a.keep_first if a.window else 0, out_scale=out_scale)
-        prompt_shaped = T >= self.tiles_min_tokens and T >= 16 * len(meta.segments)
-        if self.use_tiles:
-            # 64 tokens per CTA with the keys through shared memory, once the portion is long enough; 16 tokens per CTA for other
-            # prompt-shaped batches; the heads of a group as rows for decoding
-            if prompt_shaped and len(meta.segments) == 1 and ((T + 63) // 64) * a.heads >= self.prompt_tiles_min_ctas and \
-                    ops.seq_prompt_attention_mma_supported(self.dtype, a.dim, 0, a.vdim):
-                ops.seq_prompt_attention_mma(qf, ck, None, cv, out, meta.segments[0][1], meta.segments[0][2], window, a.scale, **kw)
-                return
-            if ops.seq_window_attention_mma_supported(self.dtype, a.dim, 0, a.vdim, a.heads, a.kv_heads, prompt_shaped):
-                ops.seq_window_attention_mma(qf, ck, None, cv, out, meta.table, window, a.scale, prompt_shaped, **kw)
-                return
-        ops.seq_window_attention(qf, None, ck, cv, out, meta.table, window, a.scale, **kw)
+        attend_window(qf, self.cache_k[i], self.cache_v[i], out, meta, a.window or FULL_WINDOW, a.scale, tiles=self.use_tiles,
+                      min_tokens=self.tiles_min_tokens, min_ctas=self.prompt_tiles_min_ctas, gate=gate, gate_per_head=True,
+                      keep_first=a.keep_first if a.window else 0, out_scale=out_scale)
 
     def _attention(self, i, m, p, h, meta, T):
         a = m.att
@@ -551,11 +539,7 @@ class LegavikModel(torch.nn.Module):
                 pair = self.buf_pair[:T * f.top * W].view(T, f.top, W)
                 ops.moe_route_grouped(h, p.router, None, idx, rw, score="softmax", groups=f.groups, keep=f.keep, group_top=GROUP_TOP,
                                       normalize=True)
-                # grouped tiles once an expert sees several rows on average; a handful of tokens stay with the row-per-CTA form
-                if self.use_tiles and T * f.top >= 4 * f.experts and ops.moe_expert_grouped_supported(h, f.ff):
-                    ops.moe_expert_grouped(h, p.gate_up, p.edown, idx, pair, f.experts, f.ff, 0.0, act="silu")
-                else:
-                    ops.moe_expert_tokens(h, p.gate_up, p.edown, idx, pair, f.experts, f.ff, 0.0, act="silu")
+                run_experts(h, p.gate_up, p.edown, idx, pair, f.experts, f.ff, tiles=self.use_tiles)
                 ops.seq_residual_tanh(x, after.alpha, after.w, after.b, y=pair, y_w=rw, x_out=x, out=h)
             if trace is not None:
                 trace.append(x.clone())
