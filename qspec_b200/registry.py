@@ -11,7 +11,7 @@ import os
 from typing import Callable, Dict
 
 _LOADERS: Dict[str, Callable] = {}
-SEQUENCE_DESIGNS = ("Mutusun", "Pitudra", "Repepel", "Kinanex", "Legavik")      # served by the sequence-mixer library alone, bfloat16 / float32
+SEQUENCE_DESIGNS = ("Mutusun", "Pitudra", "Repepel", "Kinanex", "Legavik", "Totatar")      # served by the sequence-mixer library alone, bfloat16 / float32
 _DTYPES = {"bfloat16": "bfloat16", "bf16": "bfloat16", "float32": "float32", "fp32": "float32", "float16": "float16", "fp16": "float16"}
 
 
@@ -100,6 +100,16 @@ def _load_legavik(path, cfg, dtype, device, n_slots: int = 8, max_step_tokens: i
                                         max_seq_tokens=max_seq_tokens)
 
 
+def _load_totatar(path, cfg, dtype, device, n_slots: int = 8, max_step_tokens: int = 2048, max_seq_tokens=None, **_):
+    import torch
+    from .totatar import TotatarModel
+    dt = {"bfloat16": torch.bfloat16, "float32": torch.float32, None: torch.bfloat16}.get(dtype)
+    if dt is None:
+        raise ValueError(f"Totatar runs in bfloat16 or float32, not {dtype}")
+    return TotatarModel.from_pretrained(path, dtype=dt, device=device, n_slots=n_slots, max_step_tokens=max_step_tokens,
+                                        max_seq_tokens=max_seq_tokens)
+
+
 def _load_qspec_llama(path, cfg, dtype, device, n_slots: int = 8, max_step_tokens: int = 256, **_):
     """The int4 dual-mode decoder (Llama-3 / Qwen2.5 shapes) from a Hugging Face style config.json; weights from the
     folder's QuaRot-format safetensors shards if there are any, random otherwise."""
@@ -126,5 +136,6 @@ register("Pitudra", _load_pitudra)
 register("Repepel", _load_repepel)
 register("Kinanex", _load_kinanex)
 register("Legavik", _load_legavik)
+register("Totatar", _load_totatar)
 register("LlamaForCausalLM", _load_qspec_llama)
 register("Qwen2ForCausalLM", _load_qspec_llama)
