@@ -44,14 +44,15 @@ def parse():
     ap.add_argument("--no-per-layer", action="store_true")
     ap.add_argument("--agree-shifts", default="19,20,18",
                     help="embedding shifts tried for the agree-by-construction (high-acceptance) point; '' disables it")
-    ap.add_argument("--design", default="qspec", choices=["qspec", "mutusun", "pitudra", "repepel", "kinanex", "legavik"],
+    ap.add_argument("--design", default="qspec", choices=["qspec", "mutusun", "pitudra", "repepel", "kinanex", "legavik", "totatar"],
                     help="mutusun: prefill / decode throughput and kernel rooflines of the Mutusun design next to the int4 "
                          "decoder at equal sizes; pitudra: the same for the Pitudra design next to Mutusun "
                          "(qspec_b200/bench_seq.py); repepel: the same for the Repepel design next to Pitudra "
                          "(qspec_b200/bench_repepel.py); kinanex: the same for the Kinanex design next to Pitudra "
                          "(qspec_b200/bench_kinanex.py); legavik: the same for the Legavik design next to Kinanex "
-                         "(qspec_b200/bench_legavik.py); the default workload is unchanged")
-    ap.add_argument("--sizes", default="", help="--design mutusun / pitudra / repepel / kinanex / legavik: comma-separated size names (default: all)")
+                         "(qspec_b200/bench_legavik.py); totatar: the same for the Totatar design next to Legavik "
+                         "(qspec_b200/bench_totatar.py); the default workload is unchanged")
+    ap.add_argument("--sizes", default="", help="--design mutusun / pitudra / repepel / kinanex / legavik / totatar: comma-separated size names (default: all)")
     a = ap.parse_args()
     if a.seqs is None:
         a.seqs = 32 if a.model == "70b" else 64
@@ -132,9 +133,11 @@ def cpu_reference(args, seqs, budget_s, max_samples):
 
 def main():
     args = parse()
-    if args.design in ("mutusun", "pitudra", "repepel", "kinanex", "legavik"):
+    if args.design != "qspec":
         from qspec_b200 import bench_seq
-        if args.design == "legavik":
+        if args.design == "totatar":
+            from qspec_b200.bench_totatar import run_totatar as run
+        elif args.design == "legavik":
             from qspec_b200.bench_legavik import run_legavik as run
         elif args.design == "kinanex":
             from qspec_b200.bench_kinanex import run_kinanex as run

@@ -433,10 +433,10 @@ int qspec_seq_part_norm(const float* src, const float* w, const void* gate, int 
  * q, k and v go through silu if `silu`; with conv_w (token form only) through a short causal convolution first: conv_w float32
  * [conv_c, taps] (last column: the current token), conv_b float32 [conv_c] or NULL, channel = column - conv_off, tail float32 [2][slots]
  * [taps - 1][conv_c] as for qspec_seq_conv_act. state: float32 [slots, H, D, DV], read at a segment's start (zero at position 0), written
- * at its end. seg_starts int32 [nseg]: the first rows of all segments. D <= 256.
+ * at its end. seg_starts int32 [nseg]: the first rows of all segments. D <= 1024.
  * _tokens: the segments of at most max_len tokens, token by token. _chunks: bfloat16, without convolution, the nlong segments whose first
  * rows are `starts`; chunk_rows int32 [nchunks] holds the first row of every 64 tokens of those segments, in order, chunk0 int32 [nlong]
- * the index in chunk_rows of a segment's first chunk. Section columns, ld, D and DV multiples of 8, p and state on 16-byte boundaries;
+ * the index in chunk_rows of a segment's first chunk. D <= 256; section columns, ld, D and DV multiples of 8, p and state on 16-byte boundaries;
  * scratch (bytes from the query) on 16-byte boundaries. */
 typedef struct qspec_scalar_decay_args {
   const void* p; int ld, q_off, k_off, v_off, silu;

@@ -82,16 +82,16 @@ sandwich_norm_kernel(const float* __restrict__ x_in, float* __restrict__ x_out, 
 // ---- norm of a row in equal parts, with a gate ----------------------------------------------------------------------------------
 // QSPEC_GATE_SIGMOID_AFTER: out = out_scale * unit_rms(src) * w * sigmoid(gate); QSPEC_GATE_SILU_BEFORE: out = out_scale *
 // unit_rms(src * silu(gate)) * w. unit_rms over each of `parts` equal parts. One group of TPP threads per (token, part): a warp for
-// parts of up to 1024 entries, a CTA for larger ones. Each thread's first VEC * KEEP entries stay in registers between the passes.
-template <typename T, int VEC, int TPP>
+// parts of up to 1024 entries, a CTA for larger ones. Each thread's first KEEP groups of VEC entries wait in registers with their gates
+// and weights, so that nothing is loaded after the reduction; longer rows read the rest again.
+template <typename T, int VEC, int TPP, int KEEP>
 __global__ void __launch_bounds__(256)
 part_norm_kernel(const float* __restrict__ src, const float* __restrict__ w, const T* __restrict__ gate, int gate_ld, int gate_mode,
                  T* __restrict__ out, int out_ld, long long rows, int parts, int n, float eps, float out_scale) {
   pdl_enter();
-  constexpr int KEEP = 8;
   __shared__ float red[8];
   const long long r = (long long)blockIdx.x * (256 / TPP) + threadIdx.x / TPP;
-  if (r >= rows) return;                                          // TPP = 256: one row per CTA, never taken by a part of a CTA
+  if (r >= rows) return;                                          // whole warps; TPP = 256 has one row per CTA and never leaves here
   const int l = threadIdx.x % TPP;
   const long long t = r / parts;
   const int p = (int)(r - t * parts);
@@ -100,50 +100,48 @@ part_norm_kernel(const float* __restrict__ src, const float* __restrict__ w, con
   const float* wr = w + (size_t)p * n;
   T* o = out + (size_t)t * out_ld + (size_t)p * n;
   const bool before = gate_mode == QSPEC_GATE_SILU_BEFORE;
-  auto value = [&](int c) {
-    VecF<VEC> v = ldv<VEC>(s + c);
-    if (before) {
-      const VecF<VEC> z = ldv<VEC>(g + c);
+  auto enter = [&](VecF<VEC>& v, const VecF<VEC>& z) {
+    float q = 0.f;
 #pragma unroll
-      for (int e = 0; e < VEC; ++e) v.v[e] *= silu_f(z.v[e]);
+    for (int e = 0; e < VEC; ++e) {
+      if (before) v.v[e] *= silu_act<T>(z.v[e]);
+      q += v.v[e] * v.v[e];
     }
-    return v;
+    return q;
   };
-  VecF<VEC> keep[KEEP];
-  float ss = 0.f;
+  auto leave = [&](int c, VecF<VEC> v, const VecF<VEC>& z, const VecF<VEC>& wv, float f) {
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) v.v[e] *= (before ? f : f / (1.0f + expf(-z.v[e]))) * wv.v[e];
+    stv<VEC>(o + c, v);
+  };
+  VecF<VEC> kv[KEEP], kz[KEEP], kw[KEEP];
 #pragma unroll
   for (int k = 0; k < KEEP; ++k) {
     const int c = (l + k * TPP) * VEC;
 #pragma unroll
-    for (int e = 0; e < VEC; ++e) keep[k].v[e] = 0.f;
-    if (c < n) keep[k] = value(c);
-#pragma unroll
-    for (int e = 0; e < VEC; ++e) ss += keep[k].v[e] * keep[k].v[e];
+    for (int e = 0; e < VEC; ++e) kv[k].v[e] = kz[k].v[e] = kw[k].v[e] = 0.f;
+    if (c < n) { kv[k] = ldv<VEC>(s + c); kz[k] = ldv<VEC>(g + c); kw[k] = ldv<VEC>(wr + c); }
   }
-  for (int c = (l + KEEP * TPP) * VEC; c < n; c += TPP * VEC) {
-    const VecF<VEC> v = value(c);
+  float ss = 0.f;
 #pragma unroll
-    for (int e = 0; e < VEC; ++e) ss += v.v[e] * v.v[e];
+  for (int k = 0; k < KEEP; ++k) ss += enter(kv[k], kz[k]);
+  for (int c = (l + KEEP * TPP) * VEC; c < n; c += TPP * VEC) {
+    VecF<VEC> v = ldv<VEC>(s + c);
+    ss += enter(v, ldv<VEC>(g + c));
   }
   const float sum = TPP == 32 ? warp_xor_sum(ss) : block_sum_256(ss, red);
   const float rr = out_scale / sqrtf(sum / (float)n + eps);
-  auto finish = [&](int c, VecF<VEC> v) {
-    const VecF<VEC> wv = ldv<VEC>(wr + c);
-    if (!before) {
-      const VecF<VEC> z = ldv<VEC>(g + c);
-#pragma unroll
-      for (int e = 0; e < VEC; ++e) v.v[e] *= 1.0f / (1.0f + expf(-z.v[e]));
-    }
-#pragma unroll
-    for (int e = 0; e < VEC; ++e) v.v[e] *= rr * wv.v[e];
-    stv<VEC>(o + c, v);
-  };
 #pragma unroll
   for (int k = 0; k < KEEP; ++k) {
     const int c = (l + k * TPP) * VEC;
-    if (c < n) finish(c, keep[k]);
+    if (c < n) leave(c, kv[k], kz[k], kw[k], rr);
   }
-  for (int c = (l + KEEP * TPP) * VEC; c < n; c += TPP * VEC) finish(c, value(c));
+  for (int c = (l + KEEP * TPP) * VEC; c < n; c += TPP * VEC) {
+    VecF<VEC> v = ldv<VEC>(s + c);
+    const VecF<VEC> z = ldv<VEC>(g + c);
+    enter(v, z);
+    leave(c, v, z, ldv<VEC>(wr + c), rr);
+  }
 }
 
 // ---- matrix state with one decay per head and token -------------------------------------------------------------------------------
@@ -153,8 +151,9 @@ part_norm_kernel(const float* __restrict__ src, const float* __restrict__ w, con
 // Token form: one CTA of eight warps per (segment, head, LPR * VEC value columns) walks the segment. LPR neighbouring lanes share NRW
 // neighbouring rows of the state, VEC columns each, so that whole rows are read and written; the state stays in registers from the first
 // token to the last. A token's vectors come from the projection: convolved and activated, activated, or as they are. The vectors are
-// double-buffered: two barriers per token.
-template <typename T, int NRW, int VEC, int LPR>
+// double-buffered: two barriers per token. KT > 0: a convolution of at most KT taps, whose weights and last inputs every thread keeps in
+// registers for the entries it prepares; KT = 0: filters of any length, or none.
+template <typename T, int NRW, int VEC, int LPR, int KT>
 __global__ void __launch_bounds__(256)
 scalar_decay_token_kernel(const qspec_scalar_decay_args a, int max_len) {
   pdl_enter();
@@ -186,6 +185,35 @@ scalar_decay_token_kernel(const qspec_scalar_decay_args a, int max_len) {
   float* tnew = a.conv_w ? a.tail + ((size_t)(1 - mt.phase) * a.slots + mt.slot) * K1 * C : nullptr;
   const float rate = a.A_log ? expf(a.A_log[h]) : 0.f, dtb = a.A_log ? a.dt_bias[h] : 0.f;
   const float fixed = a.A_log ? 0.f : a.decay[h], skip = a.D_skip ? a.D_skip[h] : 0.f;
+  const bool group_owner = h % rep == 0 && blockIdx.z == 0;       // writes the tail of the channels that the group's heads share
+  constexpr int NE = (2 * DP + CW + 255) / 256;
+  float hist[KT ? NE : 1][KT ? KT : 1], cwt[KT ? NE : 1][KT ? KT : 1], cbias[KT ? NE : 1];
+  int ecol[KT ? NE : 1];                                          // columns of the entries this thread prepares, -1: padding
+  if (KT) {
+#pragma unroll
+    for (int n = 0; n < NE; ++n) {
+      const int e = tid + n * 256;
+      int c = -1;
+      if (e < DP) c = e < D ? a.q_off + g * D + e : -1;
+      else if (e < 2 * DP) c = e - DP < D ? a.k_off + g * D + e - DP : -1;
+      else if (e < 2 * DP + CW) c = v0 + e - 2 * DP < DV ? a.v_off + h * DV + v0 + e - 2 * DP : -1;
+      ecol[n] = c;
+      const int ch = max(c - a.conv_off, 0);
+      cbias[n] = a.conv_b ? a.conv_b[ch] : 0.f;
+#pragma unroll
+      for (int j = 0; j < KT; ++j) {                              // leading weights of a shorter filter are zero
+        const int jr = j - (KT - a.taps);
+        const float w = a.conv_w[(size_t)ch * a.taps + max(jr, 0)];
+        cwt[n][j] = jr >= 0 ? w : 0.f;
+      }
+#pragma unroll
+      for (int j = 0; j < KT - 1; ++j) {                          // inputs before the step: position pos - (KT - 1) + j
+        const int r = j - (KT - 1 - K1);                          // row of the tail
+        const float v = K1 > 0 ? cv.told[(size_t)max(r, 0) * C + ch] : 0.f;
+        hist[n][j] = r >= 0 && mt.pos - (KT - 1) + j >= 0 ? v : 0.f;
+      }
+    }
+  }
   for (int tt = 0; tt < len; ++tt) {
     const int i = i0 + tt, pos = mt.pos + tt, buf = tt & 1;
     const T* row = (const T*)a.p + (size_t)i * a.ld;
@@ -200,7 +228,26 @@ scalar_decay_token_kernel(const qspec_scalar_decay_args a, int max_len) {
       if (a.silu) z = to_f(from_f<T>(silu_act<T>(z)));            // the activated value has the activation type, as from the convolution kernel
       return z;
     };
-    const bool group_owner = h % rep == 0 && blockIdx.z == 0;
+    if (KT) {
+#pragma unroll
+      for (int n = 0; n < NE; ++n) {
+        const int e = tid + n * 256;
+        if (e >= 2 * DP + CW) continue;
+        hist[n][KT ? KT - 1 : 0] = to_f(row[max(ecol[n], 0)]);
+        float z = cbias[n];
+#pragma unroll
+        for (int j = 0; j < KT; ++j) z += cwt[n][j] * hist[n][j];
+        if (a.silu) z = to_f(from_f<T>(silu_act<T>(z)));
+        float* dst = e < DP ? &sq[buf][e] : e < 2 * DP ? &sk[buf][e - DP] : &sv[buf][e - 2 * DP];
+        *dst = ecol[n] >= 0 ? z : 0.f;
+        if (tt == len - 1 && ecol[n] >= 0 && (e >= 2 * DP || group_owner))
+#pragma unroll
+          for (int j = 1; j < KT; ++j)
+            if (j >= KT - K1) tnew[(size_t)(j - (KT - K1)) * C + ecol[n] - a.conv_off] = hist[n][j];
+#pragma unroll
+        for (int j = 0; j + 1 < KT; ++j) hist[n][j] = hist[n][j + 1];
+      }
+    } else
     for (int e = tid; e < 2 * DP + CW; e += 256) {
       if (e < DP) sq[buf][e] = e < D ? value(a.q_off + g * D + e, group_owner) : 0.f;
       else if (e < 2 * DP) sk[buf][e - DP] = e - DP < D ? value(a.k_off + g * D + e - DP, group_owner) : 0.f;
@@ -293,17 +340,36 @@ __device__ __forceinline__ uint32_t silu_bf2(uint32_t p) {
   const __nv_bfloat162 r = __floats2bfloat162_rn(silu_act<bf16_t>(f.x), silu_act<bf16_t>(f.y));
   return *reinterpret_cast<const uint32_t*>(&r);
 }
-// 64 rows x n columns of a bfloat16 section into shared memory, eight columns per load; rows past the chunk and columns past `lim` zero
-__device__ __forceinline__ void stage_rows(bf16_t* dst, int ds, const bf16_t* src, int ld, int n, int lim, int nb, bool silu, int nthreads) {
-  const int per = n / 8;
-  for (int e = threadIdx.x; e < CHK * per; e += nthreads) {
-    const int t = e / per, c = (e - t * per) * 8;
-    uint4 v = make_uint4(0u, 0u, 0u, 0u);
-    if (t < nb && c < lim) {
-      v = *reinterpret_cast<const uint4*>(src + (size_t)t * ld + c);
-      if (silu) { v.x = silu_bf2(v.x); v.y = silu_bf2(v.y); v.z = silu_bf2(v.z); v.w = silu_bf2(v.w); }
+// 64 rows x N columns of a bfloat16 section into shared memory by 128 threads, eight columns per load; rows past the chunk and columns
+// past `lim` zero. Without silu the copies are asynchronous (the caller commits and waits); with it they pass through registers, all
+// loads of a batch before the first store.
+template <int N>
+__device__ __forceinline__ void stage_rows(bf16_t* dst, int ds, const bf16_t* src, int ld, int lim, int nb, bool silu) {
+  constexpr int PER = N / 8, TOTAL = CHK * PER / 128, BATCH = TOTAL < 8 ? TOTAL : 8;
+  if (!silu) {
+#pragma unroll
+    for (int r = 0; r < TOTAL; ++r) {
+      const int e = threadIdx.x + r * 128, t = e / PER, c = (e % PER) * 8;
+      const bool ok = t < nb && c < lim;
+      cp_async_16z(dst + t * ds + c, ok ? src + (size_t)t * ld + c : src, ok);
     }
-    *reinterpret_cast<uint4*>(dst + t * ds + c) = v;
+    return;
+  }
+#pragma unroll
+  for (int r0 = 0; r0 < TOTAL; r0 += BATCH) {
+    uint4 v[BATCH];
+#pragma unroll
+    for (int r = 0; r < BATCH; ++r) {
+      const int e = threadIdx.x + (r0 + r) * 128, t = e / PER, c = (e % PER) * 8;
+      v[r] = *reinterpret_cast<const uint4*>(src + (size_t)min(t, nb - 1) * ld + (c < lim ? c : 0));
+    }
+#pragma unroll
+    for (int r = 0; r < BATCH; ++r) {
+      const int e = threadIdx.x + (r0 + r) * 128, t = e / PER, c = (e % PER) * 8;
+      uint4 w = make_uint4(silu_bf2(v[r].x), silu_bf2(v[r].y), silu_bf2(v[r].z), silu_bf2(v[r].w));
+      if (t >= nb || c >= lim) w = make_uint4(0u, 0u, 0u, 0u);
+      *reinterpret_cast<uint4*>(dst + t * ds + c) = w;
+    }
   }
 }
 
@@ -324,32 +390,42 @@ scalar_decay_chunk_kernel(const qspec_scalar_decay_args a, const int* __restrict
   ChunkHead ch;
   ch.i0 = chunk_rows[x];
   ch.nb = min(CHK, a.meta[3 * a.ntok + ch.i0] - ch.i0);
-  chunk_decays<bf16_t>(a, ch, h, sdt, sL, &swarp);
   const bf16_t* base = (const bf16_t*)a.p + (size_t)ch.i0 * a.ld;
-  stage_rows(sk, KS, base + a.k_off + g * D, a.ld, DP, D, ch.nb, a.silu, 128);
+  const int nv = min(64, DV - v0);
+  stage_rows<DP>(sk, KS, base + a.k_off + g * D, a.ld, D, ch.nb, a.silu);
+  cp_async_commit();
+  uint4 val[4];                                                   // this thread's values, in flight during the decays
+#pragma unroll
+  for (int r = 0; r < 4; ++r) {
+    const int e = tid + r * 128, t = min(e >> 3, ch.nb - 1), c = (e & 7) * 8;
+    val[r] = *reinterpret_cast<const uint4*>(base + (size_t)t * a.ld + a.v_off + h * DV + v0 + (c < nv ? c : 0));
+  }
+  chunk_decays<bf16_t>(a, ch, h, sdt, sL, &swarp);
   __syncthreads();                                                // sL is complete
   const float end = sL[CHK - 1];
   if (tid == 0 && blockIdx.z == 0) total[(size_t)x * H + h] = expf(end);
-  const int nv = min(64, DV - v0);
-  for (int e = tid; e < CHK * 8; e += 128) {
-    const int t = e >> 3, c = (e & 7) * 8;
+#pragma unroll
+  for (int r = 0; r < 4; ++r) {
+    const int e = tid + r * 128, t = e >> 3, c = (e & 7) * 8;
     uint4 hi = make_uint4(0u, 0u, 0u, 0u), lo = hi;
     if (t < ch.nb && c < nv) {
-      uint4 v = *reinterpret_cast<const uint4*>(base + (size_t)t * a.ld + a.v_off + h * DV + v0 + c);
+      uint4 v = val[r];
       if (a.silu) { v.x = silu_bf2(v.x); v.y = silu_bf2(v.y); v.z = silu_bf2(v.z); v.w = silu_bf2(v.w); }
       const float f = expf(end - sL[t]) * sdt[t];
-      const uint32_t* vp = &v.x;
-      uint32_t* hp = &hi.x;
-      uint32_t* lp = &lo.x;
+      const uint32_t in[4] = {v.x, v.y, v.z, v.w};
+      uint32_t hp[4], lp[4];
 #pragma unroll
       for (int k = 0; k < 4; ++k) {
-        const float2 w = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(vp + k));
+        const float2 w = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&in[k]));
         tk_split_bf2(w.x * f, w.y * f, hp[k], lp[k]);
       }
+      hi = make_uint4(hp[0], hp[1], hp[2], hp[3]);
+      lo = make_uint4(lp[0], lp[1], lp[2], lp[3]);
     }
     *reinterpret_cast<uint4*>(sh + t * VS + c) = hi;
     *reinterpret_cast<uint4*>(sl + t * VS + c) = lo;
   }
+  cp_async_wait<0>();
   __syncthreads();
   const int mr = lane & 7, mm = lane >> 3;
   float* dst = add + ((size_t)x * H + h) * D * DV;
@@ -450,17 +526,31 @@ scalar_decay_out_kernel(const qspec_scalar_decay_args a, const int* __restrict__
   ch.nb = min(CHK, a.meta[3 * a.ntok + ch.i0] - ch.i0);
   const bf16_t* base = (const bf16_t*)a.p + (size_t)ch.i0 * a.ld;
   const float* src = states + ((size_t)x * H + h) * D * DV + v0;
-  for (int e = tid; e < DP * 16; e += 128) {
-    const int d = e >> 4, c = (e & 15) * 4;
-    uint4 w = make_uint4(0u, 0u, 0u, 0u);
-    if (d < D && c < nv) w = *reinterpret_cast<const uint4*>(src + (size_t)d * DV + c);
-    *reinterpret_cast<uint2*>(sh + d * VS + c) = make_uint2(__byte_perm(w.x, w.y, 0x5410), __byte_perm(w.z, w.w, 0x5410));
-    *reinterpret_cast<uint2*>(sl + d * VS + c) = make_uint2(__byte_perm(w.x, w.y, 0x7632), __byte_perm(w.z, w.w, 0x7632));
+  stage_rows<DP>(sq, KS, base + a.q_off + g * D, a.ld, D, ch.nb, a.silu);
+  stage_rows<DP>(sk, KS, base + a.k_off + g * D, a.ld, D, ch.nb, a.silu);
+  stage_rows<64>(sv, VS, base + a.v_off + h * DV + v0, a.ld, nv, ch.nb, a.silu);
+  cp_async_commit();
+#pragma unroll
+  for (int r0 = 0; r0 < DP / 8; r0 += 8) {                        // the state before the chunk, its halves apart
+    uint4 v[8];
+#pragma unroll
+    for (int r = 0; r < 8; ++r) {
+      const int e = tid + (r0 + r) * 128, d = e >> 4, c = (e & 15) * 4;
+      v[r] = *reinterpret_cast<const uint4*>(src + (size_t)min(d, D - 1) * DV + (c < nv ? c : 0));
+    }
+#pragma unroll
+    for (int r = 0; r < 8; ++r) {
+      const int e = tid + (r0 + r) * 128, d = e >> 4, c = (e & 15) * 4;
+      const bool ok = d < D && c < nv;
+      uint2 hi = make_uint2(__byte_perm(v[r].x, v[r].y, 0x5410), __byte_perm(v[r].z, v[r].w, 0x5410));
+      uint2 lo = make_uint2(__byte_perm(v[r].x, v[r].y, 0x7632), __byte_perm(v[r].z, v[r].w, 0x7632));
+      if (!ok) hi = lo = make_uint2(0u, 0u);
+      *reinterpret_cast<uint2*>(sh + d * VS + c) = hi;
+      *reinterpret_cast<uint2*>(sl + d * VS + c) = lo;
+    }
   }
-  stage_rows(sq, KS, base + a.q_off + g * D, a.ld, DP, D, ch.nb, a.silu, 128);
-  stage_rows(sk, KS, base + a.k_off + g * D, a.ld, DP, D, ch.nb, a.silu, 128);
-  stage_rows(sv, VS, base + a.v_off + h * DV + v0, a.ld, 64, nv, ch.nb, a.silu, 128);
   chunk_decays<bf16_t>(a, ch, h, sdt, sL, &swarp);
+  cp_async_wait<0>();
   __syncthreads();
   const int t0 = warp * 16, mr = lane & 7, mm = lane >> 3, ra = t0 + (lane >> 2), rb = ra + 8, cq = (lane & 3) * 2;
   if (t0 >= ch.nb) return;                                        // (uniform over the warp; no barrier follows)
@@ -590,8 +680,17 @@ static int launch_part_norm(const float* src, const float* w, const void* gate, 
                             int parts, int n, float eps, float out_scale, cudaStream_t st) {
   const long long rows = (long long)ntok * parts;
 #define PN_ARGS src, w, (const T*)gate, gate_ld, gate_mode, (T*)out, out_ld, rows, parts, n, eps, out_scale
-  if (n <= 1024) launch_pdl(part_norm_kernel<T, VEC, 32>, dim3((unsigned)((rows + 7) / 8)), dim3(256), 0, st, PN_ARGS);
-  else launch_pdl(part_norm_kernel<T, VEC, 256>, dim3((unsigned)rows), dim3(256), 0, st, PN_ARGS);
+  const int tpp = n <= 1024 ? 32 : 256, keep = (n + tpp * VEC - 1) / (tpp * VEC);
+  const dim3 grid((unsigned)((rows + 256 / tpp - 1) / (256 / tpp)));
+#define PN_KEEP(TPP)                                                                                                 \
+  do {                                                                                                               \
+    if (keep <= 2) launch_pdl(part_norm_kernel<T, VEC, TPP, 2>, grid, dim3(256), 0, st, PN_ARGS);                    \
+    else if (keep <= 4) launch_pdl(part_norm_kernel<T, VEC, TPP, 4>, grid, dim3(256), 0, st, PN_ARGS);               \
+    else launch_pdl(part_norm_kernel<T, VEC, TPP, 8>, grid, dim3(256), 0, st, PN_ARGS);                              \
+  } while (0)
+  if (tpp == 32) PN_KEEP(32);
+  else PN_KEEP(256);
+#undef PN_KEEP
 #undef PN_ARGS
   QSPEC_CHECK_LAUNCH(1);
   return QSPEC_OK;
@@ -619,7 +718,9 @@ extern "C" int qspec_seq_part_norm(const float* src, const float* w, const void*
 template <typename T, int NRW, int VEC, int LPR>
 static int launch_sd_token(const qspec_scalar_decay_args& a, int max_len, cudaStream_t st) {
   constexpr int CW = LPR * VEC;
-  launch_pdl(scalar_decay_token_kernel<T, NRW, VEC, LPR>, dim3(a.nseg, a.H, (a.DV + CW - 1) / CW), dim3(256), 0, st, a, max_len);
+  const dim3 grid(a.nseg, a.H, (a.DV + CW - 1) / CW);
+  if (NRW * LPR <= 256 && a.conv_w && a.taps <= 4) launch_pdl(scalar_decay_token_kernel<T, NRW, VEC, LPR, NRW * LPR <= 256 ? 4 : 0>, grid, dim3(256), 0, st, a, max_len);
+  else launch_pdl(scalar_decay_token_kernel<T, NRW, VEC, LPR, 0>, grid, dim3(256), 0, st, a, max_len);
   QSPEC_CHECK_LAUNCH(1);
   return QSPEC_OK;
 }
@@ -635,6 +736,10 @@ static int launch_sd_token_n(const qspec_scalar_decay_args& a, int max_len, cuda
 
 template <typename T>
 static int launch_sd_tokens(const qspec_scalar_decay_args& a, int max_len, cudaStream_t st) {
+  if (a.D > 256) {                                                // many rows: eight lanes share a row group
+    if (a.DV % 4 == 0 && ((uintptr_t)a.state & 15) == 0) return a.D <= 512 ? launch_sd_token<T, 16, 4, 8>(a, max_len, st) : launch_sd_token<T, 32, 4, 8>(a, max_len, st);
+    return a.D <= 512 ? launch_sd_token<T, 16, 1, 8>(a, max_len, st) : launch_sd_token<T, 32, 1, 8>(a, max_len, st);
+  }
   if (a.DV % 4 == 0 && ((uintptr_t)a.state & 15) == 0) {          // four columns per lane, as many lanes per row as it needs
     if (a.DV <= 32) return launch_sd_token_n<T, 4, 8>(a, max_len, st);
     if (a.DV <= 64) return launch_sd_token_n<T, 4, 16>(a, max_len, st);
@@ -676,9 +781,9 @@ extern "C" int qspec_seq_scalar_decay_chunks_supported(int ld, int q_off, int k_
 static int check_scalar_decay(const qspec_scalar_decay_args* a, int dtype) {
   QSPEC_REQUIRE(a && a->p && a->state && a->y && a->meta && a->seg_starts && (a->A_log ? (a->dt && a->dt_bias) : (a->decay && a->log_decay)),
                 QSPEC_ERR_INVALID_ARG, "seq_scalar_decay: null pointer");
-  QSPEC_REQUIRE(a->ntok >= 0 && a->nseg >= 0 && a->H > 0 && a->H <= 65535 && a->G > 0 && a->H % a->G == 0 && a->D > 0 && a->D <= 256 && a->DV > 0 &&
-                    a->DV <= 65535 * 32,
-                QSPEC_ERR_UNSUPPORTED, "seq_scalar_decay: heads %d / %d, key size %d (<= 256), value size %d", a->H, a->G, a->D, a->DV);
+  QSPEC_REQUIRE(a->ntok >= 0 && a->nseg >= 0 && a->H > 0 && a->H <= 65535 && a->G > 0 && a->H % a->G == 0 && a->D > 0 && a->D <= 1024 && a->DV > 0 &&
+                    a->DV <= 65535 * 8,
+                QSPEC_ERR_UNSUPPORTED, "seq_scalar_decay: heads %d / %d, key size %d (<= 1024), value size %d", a->H, a->G, a->D, a->DV);
   QSPEC_REQUIRE(a->q_off >= 0 && a->k_off >= 0 && a->v_off >= 0 && a->q_off + a->G * a->D <= a->ld && a->k_off + a->G * a->D <= a->ld &&
                     a->v_off + a->H * a->DV <= a->ld,
                 QSPEC_ERR_INVALID_ARG, "seq_scalar_decay: sections outside the row");

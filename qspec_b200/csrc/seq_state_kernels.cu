@@ -75,15 +75,31 @@ conv_act_run_kernel(const T* __restrict__ in, int ld, const float* __restrict__ 
   if (c >= C) return;
   const int K1 = taps - 1;
   VecF<4> rows[RUN], hist[KT], wv[KT], b;
+  const TokMeta m0 = load_meta(meta, ntok, i0);
 #pragma unroll
   for (int r = 0; r < RUN; ++r) rows[r] = ldv<4>(in + (size_t)min(i0 + r, ntok - 1) * ld + c);
+  const int first0 = m0.pos - (i0 - m0.seg_begin);
+  const bool inside = i0 - m0.seg_begin >= KT - 1;                // every input before the run lies in the step: loads without branches
+  if (inside) {
 #pragma unroll
-  for (int j = 0; j < KT; ++j)                                    // leading weights of a shorter filter are zero
+    for (int j = 0; j < KT - 1; ++j) hist[j] = ldv<4>(in + (size_t)(i0 - (KT - 1) + j) * ld + c);
+  }
+  if (taps == 4 && KT == 4 && ((uintptr_t)w & 15) == 0) {
 #pragma unroll
-    for (int e = 0; e < 4; ++e) wv[j].v[e] = j >= KT - taps ? w[(size_t)(c + e) * taps + j - (KT - taps)] : 0.f;
+    for (int e = 0; e < 4; ++e) {
+      const VecF<4> t = ldv<4>(w + (size_t)(c + e) * 4);
+#pragma unroll
+      for (int j = 0; j < KT; ++j) wv[j].v[e] = t.v[j & 3];
+    }
+  } else {
+#pragma unroll
+    for (int j = 0; j < KT; ++j)                                  // leading weights of a shorter filter are zero
+#pragma unroll
+      for (int e = 0; e < 4; ++e) wv[j].v[e] = j >= KT - taps ? w[(size_t)(c + e) * taps + j - (KT - taps)] : 0.f;
+  }
 #pragma unroll
   for (int e = 0; e < 4; ++e) b.v[e] = bias ? bias[c + e] : 0.f;
-  // input of the sequence of `mt` at position sp (before the segment's token `i`, or in it)
+  // input of the sequence of `mt` at position sp, in the step or before it
   auto get = [&](const TokMeta& mt, int first_pos, int sp) {
     VecF<4> v;
 #pragma unroll
@@ -92,31 +108,46 @@ conv_act_run_kernel(const T* __restrict__ in, int ld, const float* __restrict__ 
     else if (sp >= 0 && sp >= first_pos - K1) v = ldv<4>(tail + (((size_t)mt.phase * slots + mt.slot) * K1 + (sp - first_pos + K1)) * C + c);
     return v;
   };
+  auto emit = [&](int r) {                                        // row i0 + r from the window, which then moves on
+    hist[KT - 1] = rows[r];
+    VecF<4> acc = b;
+#pragma unroll
+    for (int j = 0; j < KT; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc.v[e] += wv[j].v[e] * hist[j].v[e];
+    if (act == QSPEC_CONV_ACT_SILU)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc.v[e] = silu_act<OT>(acc.v[e]);
+    stv<4>(out + (size_t)(i0 + r) * out_ld + c, acc);
+#pragma unroll
+    for (int j = 0; j < KT - 1; ++j) hist[j] = hist[j + 1];
+  };
+  auto write_tail = [&](const TokMeta& mt, int first_pos, int pos) {       // pos: the segment's last position
+    for (int k = 0; k < K1; ++k)
+      stv<4>(tail + (((size_t)(1 - mt.phase) * slots + mt.slot) * K1 + k) * C + c, get(mt, first_pos, pos + 1 - K1 + k));
+  };
+  if (!inside) {
+#pragma unroll
+    for (int j = 0; j < KT - 1; ++j) hist[j] = get(m0, first0, m0.pos - (KT - 1) + j);
+  }
+  if (i0 + RUN <= m0.seg_end) {                                   // one sequence's rows
+#pragma unroll
+    for (int r = 0; r < RUN; ++r) emit(r);
+    if (i0 + RUN == m0.seg_end) write_tail(m0, first0, m0.pos + RUN - 1);
+    return;
+  }
 #pragma unroll
   for (int r = 0; r < RUN; ++r) {
     const int i = i0 + r;
     if (i < ntok) {
       const TokMeta mt = load_meta(meta, ntok, i);
       const int first_pos = mt.pos - (i - mt.seg_begin);
-      if (r == 0 || i == mt.seg_begin) {
+      if (r > 0 && i == mt.seg_begin) {
 #pragma unroll
         for (int j = 0; j < KT - 1; ++j) hist[j] = get(mt, first_pos, mt.pos - (KT - 1) + j);
       }
-      hist[KT - 1] = rows[r];
-      VecF<4> acc = b;
-#pragma unroll
-      for (int j = 0; j < KT; ++j)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) acc.v[e] += wv[j].v[e] * hist[j].v[e];
-      if (act == QSPEC_CONV_ACT_SILU)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) acc.v[e] = silu_f(acc.v[e]);
-      stv<4>(out + (size_t)i * out_ld + c, acc);
-      if (i == mt.seg_end - 1)
-        for (int k = 0; k < K1; ++k)
-          stv<4>(tail + (((size_t)(1 - mt.phase) * slots + mt.slot) * K1 + k) * C + c, get(mt, first_pos, mt.pos + 1 - K1 + k));
-#pragma unroll
-      for (int j = 0; j < KT - 1; ++j) hist[j] = hist[j + 1];
+      emit(r);
+      if (i == mt.seg_end - 1) write_tail(mt, first_pos, mt.pos);
     }
   }
 }
