@@ -154,7 +154,7 @@ part_norm_kernel(const float* __restrict__ src, const float* __restrict__ w, con
 // double-buffered: two barriers per token. KT > 0: a convolution of at most KT taps, whose weights and last inputs every thread keeps in
 // registers for the entries it prepares; KT = 0: filters of any length, or none.
 template <typename T, int NRW, int VEC, int LPR, int KT>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, NRW * VEC <= 32 ? 3 : NRW * VEC <= 64 ? 2 : 1)
 scalar_decay_token_kernel(const qspec_scalar_decay_args a, int max_len) {
   pdl_enter();
   constexpr int DP = (256 / LPR) * NRW, CW = LPR * VEC;
@@ -340,16 +340,16 @@ __device__ __forceinline__ uint32_t silu_bf2(uint32_t p) {
   const __nv_bfloat162 r = __floats2bfloat162_rn(silu_act<bf16_t>(f.x), silu_act<bf16_t>(f.y));
   return *reinterpret_cast<const uint32_t*>(&r);
 }
-// 64 rows x N columns of a bfloat16 section into shared memory by 128 threads, eight columns per load; rows past the chunk and columns
+// 64 rows x N columns of a bfloat16 section into shared memory by NT threads, eight columns per load; rows past the chunk and columns
 // past `lim` zero. Without silu the copies are asynchronous (the caller commits and waits); with it they pass through registers, all
 // loads of a batch before the first store.
-template <int N>
+template <int N, int NT>
 __device__ __forceinline__ void stage_rows(bf16_t* dst, int ds, const bf16_t* src, int ld, int lim, int nb, bool silu) {
-  constexpr int PER = N / 8, TOTAL = CHK * PER / 128, BATCH = TOTAL < 8 ? TOTAL : 8;
+  constexpr int PER = N / 8, TOTAL = CHK * PER / NT, BATCH = TOTAL < 8 ? TOTAL : 8;
   if (!silu) {
 #pragma unroll
     for (int r = 0; r < TOTAL; ++r) {
-      const int e = threadIdx.x + r * 128, t = e / PER, c = (e % PER) * 8;
+      const int e = threadIdx.x + r * NT, t = e / PER, c = (e % PER) * 8;
       const bool ok = t < nb && c < lim;
       cp_async_16z(dst + t * ds + c, ok ? src + (size_t)t * ld + c : src, ok);
     }
@@ -360,12 +360,12 @@ __device__ __forceinline__ void stage_rows(bf16_t* dst, int ds, const bf16_t* sr
     uint4 v[BATCH];
 #pragma unroll
     for (int r = 0; r < BATCH; ++r) {
-      const int e = threadIdx.x + (r0 + r) * 128, t = e / PER, c = (e % PER) * 8;
+      const int e = threadIdx.x + (r0 + r) * NT, t = e / PER, c = (e % PER) * 8;
       v[r] = *reinterpret_cast<const uint4*>(src + (size_t)min(t, nb - 1) * ld + (c < lim ? c : 0));
     }
 #pragma unroll
     for (int r = 0; r < BATCH; ++r) {
-      const int e = threadIdx.x + (r0 + r) * 128, t = e / PER, c = (e % PER) * 8;
+      const int e = threadIdx.x + (r0 + r) * NT, t = e / PER, c = (e % PER) * 8;
       uint4 w = make_uint4(silu_bf2(v[r].x), silu_bf2(v[r].y), silu_bf2(v[r].z), silu_bf2(v[r].w));
       if (t >= nb || c >= lim) w = make_uint4(0u, 0u, 0u, 0u);
       *reinterpret_cast<uint4*>(dst + t * ds + c) = w;
@@ -392,7 +392,7 @@ scalar_decay_chunk_kernel(const qspec_scalar_decay_args a, const int* __restrict
   ch.nb = min(CHK, a.meta[3 * a.ntok + ch.i0] - ch.i0);
   const bf16_t* base = (const bf16_t*)a.p + (size_t)ch.i0 * a.ld;
   const int nv = min(64, DV - v0);
-  stage_rows<DP>(sk, KS, base + a.k_off + g * D, a.ld, D, ch.nb, a.silu);
+  stage_rows<DP, 128>(sk, KS, base + a.k_off + g * D, a.ld, D, ch.nb, a.silu);
   cp_async_commit();
   uint4 val[4];                                                   // this thread's values, in flight during the decays
 #pragma unroll
@@ -505,10 +505,10 @@ scalar_decay_walk_kernel(const qspec_scalar_decay_args a, const int* __restrict_
   *reinterpret_cast<float4*>(st) = S;
 }
 
-// The read-outs of a chunk: four warps of 16 tokens, 64 value columns per CTA. First q S0, whose rows are scaled by exp(L_t) in the
+// The read-outs of a chunk: eight warps of 16 tokens and 32 of the CTA's 64 value columns each. First q S0, whose rows are scaled by exp(L_t) in the
 // accumulators; then the masked, decayed scores go from the accumulators of q k^T straight into the product with the values.
 template <int DP>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(256)
 scalar_decay_out_kernel(const qspec_scalar_decay_args a, const int* __restrict__ chunk_rows, const float* __restrict__ states) {
   pdl_enter();
   extern __shared__ __align__(16) unsigned char sm_so[];
@@ -526,21 +526,21 @@ scalar_decay_out_kernel(const qspec_scalar_decay_args a, const int* __restrict__
   ch.nb = min(CHK, a.meta[3 * a.ntok + ch.i0] - ch.i0);
   const bf16_t* base = (const bf16_t*)a.p + (size_t)ch.i0 * a.ld;
   const float* src = states + ((size_t)x * H + h) * D * DV + v0;
-  stage_rows<DP>(sq, KS, base + a.q_off + g * D, a.ld, D, ch.nb, a.silu);
-  stage_rows<DP>(sk, KS, base + a.k_off + g * D, a.ld, D, ch.nb, a.silu);
-  stage_rows<64>(sv, VS, base + a.v_off + h * DV + v0, a.ld, nv, ch.nb, a.silu);
+  stage_rows<DP, 256>(sq, KS, base + a.q_off + g * D, a.ld, D, ch.nb, a.silu);
+  stage_rows<DP, 256>(sk, KS, base + a.k_off + g * D, a.ld, D, ch.nb, a.silu);
+  stage_rows<64, 256>(sv, VS, base + a.v_off + h * DV + v0, a.ld, nv, ch.nb, a.silu);
   cp_async_commit();
 #pragma unroll
-  for (int r0 = 0; r0 < DP / 8; r0 += 8) {                        // the state before the chunk, its halves apart
-    uint4 v[8];
+  for (int r0 = 0; r0 < DP / 16; r0 += 4) {                        // the state before the chunk, its halves apart
+    uint4 v[4];
 #pragma unroll
-    for (int r = 0; r < 8; ++r) {
-      const int e = tid + (r0 + r) * 128, d = e >> 4, c = (e & 15) * 4;
+    for (int r = 0; r < 4; ++r) {
+      const int e = tid + (r0 + r) * 256, d = e >> 4, c = (e & 15) * 4;
       v[r] = *reinterpret_cast<const uint4*>(src + (size_t)min(d, D - 1) * DV + (c < nv ? c : 0));
     }
 #pragma unroll
-    for (int r = 0; r < 8; ++r) {
-      const int e = tid + (r0 + r) * 128, d = e >> 4, c = (e & 15) * 4;
+    for (int r = 0; r < 4; ++r) {
+      const int e = tid + (r0 + r) * 256, d = e >> 4, c = (e & 15) * 4;
       const bool ok = d < D && c < nv;
       uint2 hi = make_uint2(__byte_perm(v[r].x, v[r].y, 0x5410), __byte_perm(v[r].z, v[r].w, 0x5410));
       uint2 lo = make_uint2(__byte_perm(v[r].x, v[r].y, 0x7632), __byte_perm(v[r].z, v[r].w, 0x7632));
@@ -552,25 +552,28 @@ scalar_decay_out_kernel(const qspec_scalar_decay_args a, const int* __restrict__
   chunk_decays<bf16_t>(a, ch, h, sdt, sL, &swarp);
   cp_async_wait<0>();
   __syncthreads();
-  const int t0 = warp * 16, mr = lane & 7, mm = lane >> 3, ra = t0 + (lane >> 2), rb = ra + 8, cq = (lane & 3) * 2;
+  const int t0 = (warp & 3) * 16, n0 = (warp >> 2) * 32, mr = lane & 7, mm = lane >> 3, ra = t0 + (lane >> 2), rb = ra + 8, cq = (lane & 3) * 2;
   if (t0 >= ch.nb) return;                                        // (uniform over the warp; no barrier follows)
-  float y[8][4], s[8][4];
+  float y[4][4], s[8][4];
 #pragma unroll
   for (int n = 0; n < 8; ++n)
 #pragma unroll
-    for (int e = 0; e < 4; ++e) { y[n][e] = 0.f; s[n][e] = 0.f; }
+    for (int e = 0; e < 4; ++e) y[n & 3][e] = s[n][e] = 0.f;
   for (int d0 = 0; d0 < D; d0 += 16) {
     uint32_t A[4], B[4];
     tk_ldmatrix_x4(A, sq + (t0 + (mm & 1) * 8 + mr) * KS + d0 + (mm >> 1) * 8);
 #pragma unroll
-    for (int n = 0; n < 8; n += 2) {
-      const int at = (d0 + (mm & 1) * 8 + mr) * VS + n * 8 + (mm >> 1) * 8;
+    for (int n = 0; n < 4; n += 2) {
+      const int at = (d0 + (mm & 1) * 8 + mr) * VS + n0 + n * 8 + (mm >> 1) * 8;
       tk_ldmatrix_x4_trans(B, sh + at);
       tk_mma_16816(y[n], A, B[0], B[1]);
       tk_mma_16816(y[n + 1], A, B[2], B[3]);
       tk_ldmatrix_x4_trans(B, sl + at);
       tk_mma_16816(y[n], A, B[0], B[1]);
       tk_mma_16816(y[n + 1], A, B[2], B[3]);
+    }
+#pragma unroll
+    for (int n = 0; n < 8; n += 2) {
       if (n * 8 <= t0 + 15) {                                     // token columns the warp's rows can see
         tk_ldmatrix_x4(B, sk + (n * 8 + (mm >> 1) * 8 + mr) * KS + d0 + (mm & 1) * 8);
         tk_mma_16816(s[n], A, B[0], B[1]);
@@ -580,7 +583,7 @@ scalar_decay_out_kernel(const qspec_scalar_decay_args a, const int* __restrict__
   }
   const float La = sL[ra], Lb = sL[rb], ea = expf(La), eb = expf(Lb);
 #pragma unroll
-  for (int n = 0; n < 8; ++n) { y[n][0] *= ea; y[n][1] *= ea; y[n][2] *= eb; y[n][3] *= eb; }
+  for (int n = 0; n < 4; ++n) { y[n][0] *= ea; y[n][1] *= ea; y[n][2] *= eb; y[n][3] *= eb; }
 #pragma unroll
   for (int j = 0; j < 4; ++j) {
     if (j * 16 > t0 + 15) break;
@@ -599,9 +602,9 @@ scalar_decay_out_kernel(const qspec_scalar_decay_args a, const int* __restrict__
       tk_split_bf2(wgt[2], wgt[3], hi[2 * u + 1], lo[2 * u + 1]);
     }
 #pragma unroll
-    for (int n = 0; n < 8; n += 2) {
+    for (int n = 0; n < 4; n += 2) {
       uint32_t B[4];
-      tk_ldmatrix_x4_trans(B, sv + (j * 16 + (mm & 1) * 8 + mr) * VS + n * 8 + (mm >> 1) * 8);
+      tk_ldmatrix_x4_trans(B, sv + (j * 16 + (mm & 1) * 8 + mr) * VS + n0 + n * 8 + (mm >> 1) * 8);
       tk_mma_16816(y[n], hi, B[0], B[1]);
       tk_mma_16816(y[n], lo, B[0], B[1]);
       tk_mma_16816(y[n + 1], hi, B[2], B[3]);
@@ -610,8 +613,8 @@ scalar_decay_out_kernel(const qspec_scalar_decay_args a, const int* __restrict__
   }
   const float skip = a.D_skip ? a.D_skip[h] : 0.f;
 #pragma unroll
-  for (int n = 0; n < 8; ++n) {
-    const int c = n * 8 + cq;
+  for (int n = 0; n < 4; ++n) {
+    const int c = n0 + n * 8 + cq;
     if (c >= nv) continue;
 #pragma unroll
     for (int u = 0; u < 2; ++u) {
@@ -764,7 +767,7 @@ static int launch_sd_chunks(const qspec_scalar_decay_args& a, const int* chunk_r
   QSPEC_CHECK_LAUNCH(1);
   launch_pdl(scalar_decay_walk_kernel, dim3((a.D * a.DV + 1023) / 1024, a.H, nlong), dim3(256), 0, st, a, starts, chunk0, add, (const float*)total);
   QSPEC_CHECK_LAUNCH(1);
-  launch_pdl(scalar_decay_out_kernel<DP>, grid, dim3(128), smem_out, st, a, chunk_rows, (const float*)add);
+  launch_pdl(scalar_decay_out_kernel<DP>, grid, dim3(256), smem_out, st, a, chunk_rows, (const float*)add);
   QSPEC_CHECK_LAUNCH(1);
   return QSPEC_OK;
 }

@@ -321,17 +321,14 @@ def _fixed(decay):
     return dict(decay=dev(torch.tensor(decay)), log_decay=dev(torch.tensor([math.log(v) if v > 0 else -1e30 for v in decay])))
 
 
-@pytest.mark.parametrize("dtype", [F32, BF16])
+@pytest.mark.parametrize("dtype,chunks", [(F32, False), (BF16, False), (BF16, True)])
 @pytest.mark.parametrize("H,D,DV", [(4, 16, 24), (3, 7, 5), (1, 64, 64), (2, 128, 96), (2, 72, 136), (1, 200, 40), (2, 256, 8), (5, 33, 130),
                                     (2, 300, 12), (1, 700, 9)])
-@pytest.mark.parametrize("chunks", [True, False])
 def test_linear_attention_with_fixed_decays(dtype, H, D, DV, chunks):
     """Portions of many lengths with the state carried over, in two sequences at a time, one of them fresh in a slot full of NaN; decays
     of one, zero and between."""
     _cuda()
     from qspec_b200 import ops
-    if chunks and dtype == F32:
-        pytest.skip("the chunk form is bfloat16")
     g = torch.Generator().manual_seed(D * DV)
     decay = [0.999, 0.5, 1.0, 0.0, 0.93][:H]
     n, m = 230, 60
@@ -384,17 +381,14 @@ def _ssm_want(cols, p, wt, H, G, N, P, act_dtype):
     return y.reshape(T, H * P)
 
 
-@pytest.mark.parametrize("dtype", [F32, BF16])
+@pytest.mark.parametrize("dtype,chunks", [(F32, False), (BF16, False), (BF16, True)])
 @pytest.mark.parametrize("H,G,N,P,taps,dt_scale", [(4, 2, 16, 24, 4, 1.0), (3, 1, 7, 5, 2, 1.0), (2, 2, 64, 64, 1, 1.0), (4, 1, 128, 32, 3, 30.0),
                                                    (2, 1, 40, 8, 6, 1.0), (6, 3, 24, 72, 4, 30.0), (1, 1, 256, 16, 4, 1.0), (2, 1, 272, 6, 3, 1.0)])
-@pytest.mark.parametrize("chunks", [True, False])
 def test_mamba2_recurrence_with_its_convolution(dtype, H, G, N, P, taps, dt_scale, chunks):
     """Portions of many lengths, down to single tokens and shorter than the filter, of two sequences; step sizes up to hundreds (decays
     far below the smallest float32); used tails and states."""
     _cuda()
     from qspec_b200 import ops
-    if chunks and dtype == F32:
-        pytest.skip("the chunk form is bfloat16")
     g = torch.Generator().manual_seed(N * P + taps)
     cols, A, wt = _ssm(g, 200, H, G, N, P, taps, dtype, dt_scale)
     B = rnd(g, 50, A.shape[1], dtype=dtype)
