@@ -15,7 +15,7 @@ from .bench_seq import SIZES, VOCAB, _throughput, _time_us
 # the sizes of `bench_legavik.LEGAVIK_SIZES` (width, heads x 128, key/value heads, window, experts) with a dense feed-forward size, a shared
 # expert as large as a routed one, and a Mamba-2 mixer of twice the width: heads of 64, a state of 128, eight groups
 TOTATAR_SIZES = {
-    n: dict({k: v for k, v in s.items() if k not in ("rank", "groups", "keep_first", "latent")}, ff=SIZES[n]["ff"], shared=s["moe"][1],
+    n: dict({k: v for k, v in s.items() if k not in ("rank", "groups", "keep_first", "latent", "side")}, ff=SIZES[n]["ff"], shared=s["moe"][1],
             ssm=(2 * s["width"] // 64, 8, 128, 64)) for n, s in bench_legavik.LEGAVIK_SIZES.items()
 }
 

@@ -219,7 +219,7 @@ def _attend(form, q, ck, cv, out, meta, window, scale, **kw):
         ops.seq_window_attention_mma(q, ck, None, cv, out, meta.table, window, scale, form == "rows", **kw)
 
 
-FORMS = [("plain", F32, (4, 2, 12, 10)), ("plain", F32, (3, 1, 96, 64)), ("plain", BF16, (5, 1, 96, 33)), ("heads", BF16, (8, 1, 64, 64)),
+FORMS = [("plain", F32, (4, 2, 12, 10)), ("plain", F32, (3, 1, 80, 56)), ("plain", BF16, (5, 1, 112, 33)), ("heads", BF16, (8, 1, 64, 64)),
          ("heads", BF16, (4, 2, 128, 64)), ("rows", BF16, (4, 2, 64, 128)), ("tile", BF16, (2, 1, 64, 64)), ("tile", BF16, (2, 1, 128, 128))]
 
 
